@@ -146,6 +146,14 @@ def _register_nudusun():
 _register_nudusun()
 
 
+def _register_ramopel():
+    from .ramopel import RamopelConfig, ramopel_plan
+    register_architecture("Ramopel", RamopelConfig.from_dict, ramopel_plan)
+
+
+_register_ramopel()
+
+
 def _register_kizezen():
     from .kizezen import KizezenConfig, kizezen_plan
     register_architecture("Kizezen", KizezenConfig.from_dict, kizezen_plan)

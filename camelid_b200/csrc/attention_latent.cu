@@ -6,8 +6,9 @@
 //   out_h(i)      = Uv_h (sum_j w_ij c_j)
 //
 // so the cache holds rows [c_j, t_j] of C + R channels, one "key head" for all query heads, whose first C channels are
-// the values as well; the attention itself is the library's general kernel (attention_window.cu). Here: the kernel that
-// prepares a step's rows, and the product per head that applies Uk_h^T to the queries and Uv_h to the outputs.
+// the values as well; the attention itself is the library's general kernel (attention_window.cu) or, in bfloat16, the
+// tensor-core kernel below; both take a window. Here also: the kernel that prepares a step's rows, and the product per
+// head that applies Uk_h^T to the queries and Uv_h to the outputs.
 #include "common.cuh"
 
 // 16-byte asynchronous copies into shared memory, matrix fragments out of it, and the bfloat16 tensor-core instruction
@@ -47,8 +48,12 @@ __device__ __forceinline__ uint32_t la_pack(float lo, float hi) {
 
 
 // proj [rows, ld] float (n_splits matrices split_stride apart, added in split order): q (heads x (D + R), head by head
-// [plain D, turned R]), then C + R columns of the down projection, then `extra` columns (an output gate's logits).
+// [plain D, turned R]), then Q columns of a latent that the queries are made from, then C + R columns of the down
+// projection (where has_down), then `extra` columns (an output gate's logits). Any of them may be missing (heads 0, Q 0,
+// has_down 0): queries that go through a latent come in a second launch, and a layer that reads another layer's rows
+// has no down projection.
 // One block per row:
+//   cq [rows, Q]                        rmsnorm(query latent) * wq, compute type
 //   q_plain [rows, heads x D]           the unturned query parts, compute type
 //   q_full  [rows, heads x (C + R)]     the turned parts, at channels C.. of every head (the first C are written later)
 //   k_pages [pages, 1, 64, C + R]       [rmsnorm(down[:C]) * w, turned(down[C:])]
@@ -60,16 +65,17 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float* __rest
                                                              const float* __restrict__ inv_freq, int pairing, float amp,
                                                              const int* __restrict__ row_seq, const int* __restrict__ row_pos,
                                                              const int* __restrict__ table, int max_blocks, T* __restrict__ q_plain,
-                                                             T* __restrict__ q_full, T* __restrict__ k_pages, int heads, int D, int R, int C) {
-    __shared__ float red[32];
+                                                             T* __restrict__ q_full, T* __restrict__ k_pages, int heads, int D, int R, int C,
+                                                             int has_down, int Q, const TW* __restrict__ cq_w, T* __restrict__ cq) {
+    __shared__ float red[32], red_q[32];
     __shared__ float2 turn[128];
     extern __shared__ __align__(16) float x[];
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.x;
-    const int qw = heads * (D + R), total = qw + C + R + extra;
+    const int q_at = heads * (D + R), qw = q_at + Q, total = qw + (has_down ? C + R : 0) + extra;     // qw: where the down columns start
     const float* src = proj + (size_t)r * ld;
-    float ss = 0.f;
+    float ss = 0.f, ssq = 0.f;
     for (int c = threadIdx.x; c < total; c += blockDim.x) {
         float v = src[c];
         for (int s0 = 1; s0 < n_splits; s0 += 8) {
@@ -80,16 +86,21 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float* __rest
             for (int k = 0; k < 8; ++k) v += s0 + k < n_splits ? t[k] : 0.f;
         }
         x[c] = v;
-        if (c >= qw && c < qw + C) ss = fmaf(v, v, ss);
+        if (has_down && c >= qw && c < qw + C) ss = fmaf(v, v, ss);
+        if (c >= q_at && c < qw) ssq = fmaf(v, v, ssq);
     }
     const int pos = row_pos[r];
-    const int page = table[(size_t)row_seq[r] * max_blocks + pos / CML_PAGE];
+    const int page = has_down ? table[(size_t)row_seq[r] * max_blocks + pos / CML_PAGE] : -1;
     for (int i = threadIdx.x; i < R / 2; i += blockDim.x) {
         float sn, cs;
         sincosf((float)pos * inv_freq[i], &sn, &cs);
         turn[i] = make_float2(cs * amp, sn * amp);
     }
     const float c_scale = 1.0f / sqrtf(block_sum(ss, red) / (float)C + eps);       // (has the barrier that x and turn need)
+    if (Q > 0) {
+        const float q_scale = 1.0f / sqrtf(block_sum(ssq, red_q) / (float)Q + eps);
+        for (int c = threadIdx.x; c < Q; c += blockDim.x) cq[(size_t)r * Q + c] = from_f32<T>(x[q_at + c] * q_scale * to_f32(cq_w[c]));
+    }
     for (int c = threadIdx.x; c < extra; c += blockDim.x) extra_out[(size_t)r * extra + c] = x[total - extra + c];
     const int half = R / 2;
     // channel e of a turned part that starts at xs
@@ -117,10 +128,12 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const float* __rest
 extern "C" int cml_latent_prepare(const float* proj, long ld, int n_splits, long split_stride, int extra, float* extra_out,
                                   const void* c_w, int w_dtype, float eps, const float* inv_freq, int pairing, float amp,
                                   const int* row_seq, const int* row_pos, const int* table, int max_blocks, void* q_plain,
-                                  void* q_full, void* k_pages, int dtype, int rows, int heads, int D, int R, int C, void* stream) {
+                                  void* q_full, void* k_pages, int dtype, int rows, int heads, int D, int R, int C, int has_down, int Q,
+                                  const void* cq_w, void* cq, void* stream) {
     if (rows <= 0) return 0;
-    if (R < 0 || R > 256 || (R & 1) || C < 1 || D < 0 || n_splits < 1 || extra < 0) return CML_ERR_BAD_SIZE;
-    const size_t smem = (size_t)(heads * (D + R) + C + R + extra + 4) * sizeof(float);
+    if (R < 0 || R > 256 || (R & 1) || C < 1 || D < 0 || n_splits < 1 || extra < 0 || heads < 0 || Q < 0) return CML_ERR_BAD_SIZE;
+    if ((has_down && (!c_w || !k_pages)) || (Q && (!cq_w || !cq)) || (heads && (!q_full || !q_plain))) return CML_ERR_BAD_SIZE;
+    const size_t smem = (size_t)(heads * (D + R) + Q + (has_down ? C + R : 0) + extra + 4) * sizeof(float);
     if (smem > 200 * 1024) return CML_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
 #define LP_CASE(T_, TW_, D_, DW_)                                                                                               \
@@ -128,7 +141,7 @@ extern "C" int cml_latent_prepare(const float* proj, long ld, int n_splits, long
         if (smem > 48 * 1024 && cml_allow_smem<latent_prepare_kernel<T_, TW_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE;   \
         launch_pdl(latent_prepare_kernel<T_, TW_>, dim3(rows), dim3(256), smem, s, proj, ld, n_splits, split_stride, extra,     \
                    extra_out, (const TW_*)c_w, eps, inv_freq, pairing, amp, row_seq, row_pos, table, max_blocks, (T_*)q_plain,  \
-                   (T_*)q_full, (T_*)k_pages, heads, D, R, C);                                                                  \
+                   (T_*)q_full, (T_*)k_pages, heads, D, R, C, has_down, Q, (const TW_*)cq_w, (T_*)cq);                          \
         return cml_launch_status();                                                                                             \
     }
     LP_CASE(float, float, CML_DTYPE_F32, CML_DTYPE_F32)
@@ -372,6 +385,7 @@ struct LatentPromptParams {
     const float* gate; long gate_ld; int gate_col;      // float [rows, gate_ld] or null: one logit per head
     int heads, C, R;
     float scale;
+    int window;             // a row sees itself and the window - 1 positions before it; 0: every earlier position
     // single tokens over long contexts: a sequence's pages are dealt to gridDim.y blocks, `tiles_per_split` pages each; every
     // block leaves its rows' maximum (scaled), sum and unnormalised sums as floats in `partial`
     // [split, row, head, 2 + C], and a second kernel merges them (and adds the sink's term and the gate)
@@ -398,7 +412,9 @@ __global__ void __launch_bounds__(256, 1) latent_prompt_kernel(const LatentPromp
     const int start = p.seq_start[seq], n_new = p.seq_new[seq], row0 = p.seq_row0[seq];
     const int tokens = min(p.tokens_per_tile, n_new - q0);
     const int all_key_tiles = (start + q0 + tokens + LA_KEYS - 1) / LA_KEYS;
-    const int t_begin = p.partial ? min((int)blockIdx.y * p.tiles_per_split, all_key_tiles) : 0;
+    // the first page that the tile's first token (the one with the oldest view) still sees
+    const int first_tile = p.window > 0 ? max(0, start + q0 - p.window + 1) / LA_KEYS : 0;
+    const int t_begin = p.partial ? min(first_tile + (int)blockIdx.y * p.tiles_per_split, all_key_tiles) : first_tile;
     const int n_key_tiles = p.partial ? min(t_begin + p.tiles_per_split, all_key_tiles) : all_key_tiles;
     const int* tb = p.table + (size_t)seq * p.max_blocks;
     const int chunks16 = D / 8;                                    // 16-byte pieces of a row
@@ -443,7 +459,7 @@ __global__ void __launch_bounds__(256, 1) latent_prompt_kernel(const LatentPromp
     const int n_groups = p.C / 32;                                 // groups of 16 channels in a half
     const int ch0 = half * (p.C / 2);
     // the two rows a lane holds pieces of: wrow + lane / 4 and that + 8
-    int pos[2];
+    int pos[2], low[2];                                            // the newest and the oldest key each of them sees
     bool valid[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -451,6 +467,7 @@ __global__ void __launch_bounds__(256, 1) latent_prompt_kernel(const LatentPromp
         const int tok = r / HB, hd = chunk * HB + r % HB;
         valid[h] = tok < tokens && hd < p.heads;
         pos[h] = valid[h] ? start + q0 + tok : 0x7fffffff;         // rows that stand for nothing see everything: no empty softmax
+        low[h] = valid[h] && p.window > 0 ? start + q0 + tok - p.window + 1 : 0;
     }
     float o[NG][2][4];
 #pragma unroll
@@ -501,13 +518,14 @@ __global__ void __launch_bounds__(256, 1) latent_prompt_kernel(const LatentPromp
         // mask and maximum per row: a row's 32 scores lie in the four lanes of a quad, the other 32 with the partner
         const int key0 = t * LA_KEYS + kb + 2 * (lane & 3);
         float mx[2] = {-INFINITY, -INFINITY};
-        const bool page_whole = (t + 1) * LA_KEYS - 1 <= start + q0;      // every row of the tile sees all of this page
+        // every row of the tile sees all of this page
+        const bool page_whole = (t + 1) * LA_KEYS - 1 <= start + q0 && (p.window <= 0 || t * LA_KEYS > start + q0 + tokens - 1 - p.window);
 #pragma unroll
         for (int n = 0; n < 4; ++n)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + 8 * n + (e & 1), h = e >> 1;
-                if (!page_whole && key > pos[h]) s[n][e] = -INFINITY;
+                if (!page_whole && (key > pos[h] || key < low[h])) s[n][e] = -INFINITY;
                 mx[h] = fmaxf(mx[h], s[n][e]);
             }
 #pragma unroll
@@ -521,7 +539,7 @@ __global__ void __launch_bounds__(256, 1) latent_prompt_kernel(const LatentPromp
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             mx[h] = fmaxf(mx[h], mx_other[h]);
-            const float m_new = fmaxf(m[h], mx[h]);                // finite from a sequence's first page on: key 0 is visible to every row
+            const float m_new = fmaxf(m[h], mx[h]);                // (minus infinity while a row's window has not begun)
             corr[h] = m[h] == -INFINITY ? 0.f : exp2f((m[h] - m_new) * sl2);
             m[h] = m_new;
         }
@@ -676,8 +694,9 @@ extern "C" int cml_latent_prompt(const void* q, const void* k_pages, void* out, 
                                  const int* tile_seq, const int* tile_q0, int n_tiles, int tokens_per_tile, const int* seq_row0,
                                  const int* seq_start, const int* seq_new, const float* sink, const float* gate, long gate_ld,
                                  int gate_col, int heads, int C, int R, float scale, float* partial, int n_splits,
-                                 int tiles_per_split, long rows_total, void* stream) {
+                                 int tiles_per_split, long rows_total, int window, void* stream) {
     if (n_tiles <= 0) return 0;
+    if (window < 0) return CML_ERR_BAD_SIZE;
     if (partial != nullptr && (n_splits < 1 || n_splits > 65535 || tiles_per_split < 1 || tokens_per_tile != 1)) return CML_ERR_BAD_SIZE;
     if (heads < 1 || C < 32 || (C & 31) || (R & 15) || C > 512 || R < 0) return CML_ERR_BAD_SIZE;
     const int HB = heads < LA_ROWS ? heads : LA_ROWS;
@@ -689,7 +708,7 @@ extern "C" int cml_latent_prompt(const void* q, const void* k_pages, void* out, 
     p.q = (const bf16*)q; p.k_pages = (const bf16*)k_pages; p.out = (bf16*)out; p.table = table; p.max_blocks = max_blocks;
     p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.n_tiles = n_tiles; p.tokens_per_tile = tokens_per_tile;
     p.seq_row0 = seq_row0; p.seq_start = seq_start; p.seq_new = seq_new; p.sink = sink; p.gate = gate; p.gate_ld = gate_ld;
-    p.gate_col = gate_col; p.heads = heads; p.C = C; p.R = R; p.scale = scale;
+    p.gate_col = gate_col; p.heads = heads; p.C = C; p.R = R; p.scale = scale; p.window = window;
     p.partial = partial; p.tiles_per_split = tiles_per_split; p.rows_total = rows_total;
     const size_t smem = (size_t)(LA_ROWS + 2 * LA_KEYS) * ((C + R) * 2 + 16) + 8 * 2 * 4 * 32 * sizeof(uint32_t);
     if (smem > 227 * 1024) return CML_ERR_BAD_SIZE;

@@ -26,10 +26,12 @@
 // for the choice alone, and with n_groups > 1 the experts form n_groups equal groups of neighbours of which only
 // the `keep_groups` with the largest choice score of any member stay open (the others' choice scores count as
 // minus infinity). The weights are the chosen experts' uncorrected scores times `weight_scale`.
+// `bias` [E] (may be null) is added to the logits themselves, so it counts for the choice and for the weights.
 // Shared memory per warp: the scores (E floats), the choice scores (E floats), the groups' best (n_groups floats).
 __global__ void route_topk_kernel(const float* __restrict__ logits, long ld, int n_splits, long split_stride, int rows, int E,
                                   int top, int score_mode, int renorm, const float* __restrict__ correction, int n_groups,
-                                  int keep_groups, float weight_scale, int* __restrict__ ids, float* __restrict__ wts) {
+                                  int keep_groups, float weight_scale, int* __restrict__ ids, float* __restrict__ wts,
+                                  const float* __restrict__ bias) {
     extern __shared__ float rt_z[];
     pdl_wait();
     pdl_launch_dependents();
@@ -49,7 +51,7 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, long ld, int
 #pragma unroll
             for (int k = 0; k < 8; ++k) v += s0 + k < n_splits ? t[k] : 0.f;
         }
-        z[e] = v;
+        z[e] = bias ? v + bias[e] : v;
     }
     __syncwarp();
     float zmax = -INFINITY, zsum = 0.f;
@@ -118,14 +120,14 @@ __global__ void route_topk_kernel(const float* __restrict__ logits, long ld, int
 
 extern "C" int cml_route_topk(const float* logits, long ld, int n_splits, long split_stride, int rows, int E, int top,
                               int score_mode, int renorm, const float* correction, int n_groups, int keep_groups,
-                              float weight_scale, int* ids, float* wts, void* stream) {
+                              float weight_scale, int* ids, float* wts, const float* bias, void* stream) {
     if (rows <= 0) return 0;
     if (E < 1 || E > 1024 || top < 1 || top > E || n_splits < 1) return CML_ERR_BAD_SIZE;
     if (n_groups < 1 || E % n_groups || keep_groups < 1 || keep_groups > n_groups) return CML_ERR_BAD_SIZE;
     const bool separate = correction != nullptr || n_groups > 1;
     const size_t smem = (size_t)4 * (separate ? 2 * E + n_groups : E) * sizeof(float);
     launch_pdl(route_topk_kernel, dim3((rows + 3) / 4), dim3(128), smem, (cudaStream_t)stream, logits, ld,
-               n_splits, split_stride, rows, E, top, score_mode, renorm, correction, n_groups, keep_groups, weight_scale, ids, wts);
+               n_splits, split_stride, rows, E, top, score_mode, renorm, correction, n_groups, keep_groups, weight_scale, ids, wts, bias);
     return cml_launch_status();
 }
 
@@ -339,17 +341,26 @@ extern "C" int cml_expert_gemm(const void* A, const void* W, const void* W2, int
     return cml_launch_status();
 }
 
-// out[row] = sum over splits of shared[split][row] + sum over the row's choices, in their order, of y[pos] (* weight).
+// out[row] (+)= sum over splits of shared[split][row] (* gate) + sum over the row's choices, in their order, of y[pos] (* weight).
+// `shared_gate` (may be null): one logit per row (n_gate split sums gate_stride apart, rows gate_ld apart) whose sigmoid
+// multiplies the shared expert's row. `accumulate`: add to what `out` holds (the residual stream).
 // A choice of an identity expert (ids >= real_experts; `ids` may be null: there are none) adds the row itself
 // (`same` [rows, hidden], float or the compute type) times its weight.
 template <typename TS>
 __global__ void expert_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of_pair, const float* __restrict__ wts,
                                       int top, int scale_output, const float* __restrict__ shared, int shared_splits,
                                       long shared_stride, const int* __restrict__ ids, int real_experts,
-                                      const TS* __restrict__ same, float* __restrict__ out, int hidden) {
+                                      const TS* __restrict__ same, float* __restrict__ out, int hidden,
+                                      const float* __restrict__ shared_gate, long gate_ld, int n_gate, long gate_stride, int accumulate) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.x;
+    float sg = 1.0f;
+    if (shared_gate) {
+        float z = 0.f;
+        for (int s = 0; s < n_gate; ++s) z += shared_gate[(size_t)s * gate_stride + (size_t)r * gate_ld];
+        sg = 1.0f / (1.0f + expf(-z));
+    }
     if ((hidden & 3) == 0) {                                    // four columns a thread, 16-byte accesses
         for (int c = threadIdx.x * 4; c < hidden; c += blockDim.x * 4) {
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -357,6 +368,7 @@ __global__ void expert_combine_kernel(const float* __restrict__ y, const int* __
                 const float4 t = *reinterpret_cast<const float4*>(shared + (size_t)s * shared_stride + (size_t)r * hidden + c);
                 v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
             }
+            if (shared_gate) { v.x *= sg; v.y *= sg; v.z *= sg; v.w *= sg; }
             for (int k = 0; k < top; ++k) {
                 const int p = r * top + k;
                 const bool ident = ids != nullptr && ids[p] >= real_experts;
@@ -370,34 +382,40 @@ __global__ void expert_combine_kernel(const float* __restrict__ y, const int* __
                 const float w = (scale_output || ident) ? wts[p] : 1.0f;
                 v.x += t.x * w; v.y += t.y * w; v.z += t.z * w; v.w += t.w * w;
             }
-            *reinterpret_cast<float4*>(out + (size_t)r * hidden + c) = v;
+            float4* o = reinterpret_cast<float4*>(out + (size_t)r * hidden + c);
+            if (accumulate) { const float4 t = *o; v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w; }
+            *o = v;
         }
         return;
     }
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
         float v = 0.f;
         for (int s = 0; s < shared_splits; ++s) v += shared[(size_t)s * shared_stride + (size_t)r * hidden + c];
+        if (shared_gate) v *= sg;
         for (int k = 0; k < top; ++k) {
             const int p = r * top + k;
             const bool ident = ids != nullptr && ids[p] >= real_experts;
             const float t = ident ? to_f32(same[(size_t)r * hidden + c]) : y[(size_t)pos_of_pair[p] * hidden + c];
             v += (scale_output || ident) ? t * wts[p] : t;
         }
-        out[(size_t)r * hidden + c] = v;
+        out[(size_t)r * hidden + c] = accumulate ? out[(size_t)r * hidden + c] + v : v;
     }
 }
 
 extern "C" int cml_expert_combine(const float* y, const int* pos_of_pair, const float* wts, int top, int scale_output,
                                   const float* shared, int shared_splits, long shared_stride, const int* ids, int real_experts,
-                                  const void* same, int same_dtype, float* out, int rows, int hidden, void* stream) {
+                                  const void* same, int same_dtype, float* out, int rows, int hidden, const float* shared_gate,
+                                  long gate_ld, int n_gate, long gate_stride, int accumulate, void* stream) {
     if (rows <= 0) return 0;
     if (ids != nullptr && same == nullptr) return CML_ERR_BAD_SIZE;
     const dim3 block(hidden >= 1024 ? 256 : 128);
     if (same_dtype == CML_DTYPE_BF16)
         launch_pdl(expert_combine_kernel<bf16>, dim3(rows), block, 0, (cudaStream_t)stream, y, pos_of_pair, wts, top,
-                   scale_output, shared, shared ? shared_splits : 0, shared_stride, ids, real_experts, (const bf16*)same, out, hidden);
+                   scale_output, shared, shared ? shared_splits : 0, shared_stride, ids, real_experts, (const bf16*)same, out, hidden,
+                   shared_gate, gate_ld, n_gate, gate_stride, accumulate);
     else
         launch_pdl(expert_combine_kernel<float>, dim3(rows), block, 0, (cudaStream_t)stream, y, pos_of_pair, wts, top,
-                   scale_output, shared, shared ? shared_splits : 0, shared_stride, ids, real_experts, (const float*)same, out, hidden);
+                   scale_output, shared, shared ? shared_splits : 0, shared_stride, ids, real_experts, (const float*)same, out, hidden,
+                   shared_gate, gate_ld, n_gate, gate_stride, accumulate);
     return cml_launch_status();
 }

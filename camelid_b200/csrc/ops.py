@@ -24,7 +24,7 @@ _SIGNATURES = {
     ("rowwise", "cml_embed_positions"): [c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
                                          c_int, c_int, c_void_p, c_void_p],
     ("rowwise", "cml_rmsnorm"): [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p,
-                                 c_int, c_long, c_void_p],
+                                 c_int, c_long, c_void_p, c_void_p, c_void_p],
     ("rowwise", "cml_add_partials"): [c_void_p, c_void_p, c_int, c_long, c_void_p],
     ("rowwise", "cml_swiglu_packed"): [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("rope_kv", "cml_rope_kv_write"): [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
@@ -125,8 +125,12 @@ _SIGNATURES = {
     ("recurrence", "cml_memory_scan"): [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                                         c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                         c_int, c_int, c_int, c_void_p],
-    ("recurrence", "cml_head_norm_gate"): [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_long, c_int, c_void_p, c_int,
-                                           c_int, c_int, c_int, c_float, c_int, c_void_p],
+    ("recurrence", "cml_head_norm_gate"): [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_long, c_int, c_void_p, c_long,
+                                           c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    ("recurrence", "cml_delta_inputs"): [c_void_p, c_long, c_int, c_long, c_void_p, c_int, c_long, c_void_p, c_int, c_int, c_void_p,
+                                         c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    ("recurrence", "cml_general_delta_scan"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                               c_int, c_int, c_int, c_int, c_void_p],
     ("attention_window", "cml_qk_norm_kv_write"): [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p,
                                                    c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                                    c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -139,19 +143,23 @@ _SIGNATURES = {
                                               c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
     ("attention_latent", "cml_latent_prepare"): [c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p,
                                                  c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                                                 c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                                 c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                                                 c_void_p],
     ("attention_latent", "cml_head_product"): [c_void_p, c_long, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int,
                                                c_int, c_void_p],
     ("attention_latent", "cml_latent_prompt"): [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_int,
-                                                c_int, c_float, c_void_p, c_int, c_int, c_long, c_void_p],
+                                                c_int, c_float, c_void_p, c_int, c_int, c_long, c_int, c_void_p],
     ("recurrence", "cml_retention_scan"): [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrence", "cml_rotate_rows"): [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
                                         c_int, c_float, c_void_p],
+    ("token_ops", "cml_tanh_columns"): [c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+    ("token_ops", "cml_poly_norm"): [c_void_p, c_int, c_long, c_long, c_void_p, c_int, c_void_p, c_float, c_void_p, c_long, c_int,
+                                     c_int, c_void_p],
     ("token_ops", "cml_scale_values"): [c_void_p, c_long, c_float, c_void_p],
     ("experts", "cml_route_topk"): [c_void_p, c_long, c_int, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
-                                    c_float, c_void_p, c_void_p, c_void_p],
+                                    c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     ("experts", "cml_expert_plan"): [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     ("gemm_tc", "cml_gemm_tc_grouped"): [c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_long, c_int,
                                          c_int, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -160,7 +168,8 @@ _SIGNATURES = {
     ("experts", "cml_expert_gemm"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
                                      c_void_p, c_void_p],
     ("experts", "cml_expert_combine"): [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_long, c_void_p, c_int,
-                                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+                                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_long, c_int, c_long, c_int,
+                                        c_void_p],
     ("random_fill", "cml_random_fill"): [c_void_p, c_int, ctypes.c_longlong, ctypes.c_ulonglong, ctypes.c_ulonglong,
                                          ctypes.c_double, ctypes.c_double, c_void_p],
 }
@@ -331,11 +340,14 @@ def embed_positions(table: torch.Tensor, tokens: torch.Tensor, scale: float, pos
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, rows_index: torch.Tensor | None = None,
-            partial: torch.Tensor | None = None):
+            partial: torch.Tensor | None = None, weight2=None, out2=None):
     """out[r] = rmsnorm(x[rows_index[r] or r]) * weight; x float32, out float32 or bfloat16.
     ``partial`` (float32 [splits, x rows, hidden]) is first added to x, split by split; without
-    ``rows_index`` the sum is written back to x."""
-    _dev(x, weight, out, rows_index, partial)
+    ``rows_index`` the sum is written back to x. ``weight2`` / ``out2``: a second norm of the same rows that differs in
+    its weight alone, out of the same pass."""
+    _dev(x, weight, out, rows_index, partial, weight2, out2)
+    assert weight2 is None or (weight2.dtype == weight.dtype and weight2.shape == weight.shape and out2.dtype == out.dtype
+                               and out2.shape == out.shape and out2.is_contiguous())
     rows, hidden = out.shape
     assert x.dtype == torch.float32 and x.shape[1] == hidden and weight.shape[0] == hidden
     assert x.is_contiguous() and out.is_contiguous()
@@ -347,7 +359,7 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
         n_splits, stride = partial.shape[0], partial.stride(0)
     _check(_fn("rowwise", "cml_rmsnorm")(_p(x), _p(weight), dtype_code(weight.dtype), _p(out), dtype_code(out.dtype),
                                         _p(rows_index), rows, hidden, float(eps), _p(partial), n_splits, stride,
-                                        _stream()), "rmsnorm")
+                                        _p(weight2), _p(out2), _stream()), "rmsnorm")
 
 
 def add_partials(x: torch.Tensor, partial: torch.Tensor):
@@ -511,6 +523,33 @@ def bias_act_(x: torch.Tensor, bias, act: int):
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == x.shape[1] and bias.is_contiguous())
     _check(_fn("token_ops", "cml_bias_act")(_p(x), dtype_code(x.dtype), _p(bias), x.shape[0], x.shape[1], int(act), _stream()),
            "bias_act")
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor):
+    """out = a N(z) + b N(z^2) + c N(z^3) + e with N(y) = y / sqrt(mean(y^2) + eps) over a row and (a, b, c, e) = ``coef``
+    (float32 [4]). ``z``: float32 split sums [splits, rows, n] that are added first, or rows [rows, n] of ``out``'s type,
+    which may be ``out`` itself; ``out`` [rows, n], rows any stride."""
+    _dev(z, coef, out)
+    rows, width = out.shape
+    assert coef.dtype == torch.float32 and coef.numel() == 4 and out.stride(1) == 1
+    assert z.shape[-2:] == out.shape and z.stride(-1) == 1
+    split = z.dim() == 3
+    assert z.dtype == (torch.float32 if split else out.dtype)
+    _check(_fn("token_ops", "cml_poly_norm")(_p(z) if split else None, z.shape[0] if split else 0, z.stride(0) if split else 0,
+                                             z.stride(-2), None if split else _p(z), dtype_code(out.dtype), _p(coef), float(eps),
+                                             _p(out), out.stride(0), rows, width, _stream()), "poly_norm")
+
+
+def tanh_columns(z: torch.Tensor, col0: int, out: torch.Tensor):
+    """out[r, c] = tanh(z[r, col0 + c]) in the compute type; ``z`` float32 [rows, n] or split sums [splits, rows, n] that
+    are added first; ``out`` [rows, columns] contiguous."""
+    _dev(z, out)
+    if z.dim() == 2:
+        z = z.unsqueeze(0)
+    assert z.dtype == torch.float32 and z.stride(2) == 1 and z.shape[1] == out.shape[0] and col0 + out.shape[1] <= z.shape[2]
+    assert out.is_contiguous()
+    _check(_fn("token_ops", "cml_tanh_columns")(_p(z), z.stride(1), z.shape[0], z.stride(0), int(col0), _p(out), dtype_code(out.dtype),
+                                                out.shape[0], out.shape[1], _stream()), "tanh_columns")
 
 
 def gate_rows_(x: torch.Tensor, gate: torch.Tensor, gate_col: int):
@@ -698,16 +737,60 @@ def head_norm_gate(raw: torch.Tensor, with_den: bool, w: torch.Tensor, w_per_hea
                    out: torch.Tensor, heads: int, value_dim: int, eps: float, gate_silu: bool = False):
     """Per (row, head): the scan's output (divided by its denominator where it carries one), RMS
     norm over value_dim, times ``w`` (float32 [value_dim] or [heads * value_dim]; None: no weight) and
-    sigmoid(gate[:, gate_col + ...]) (``gate_silu``: times silu of it); ``out`` [rows, heads * value_dim] in the compute type."""
+    sigmoid(gate[:, gate_col + ...]) (``gate_silu``: times silu of it); ``out`` [rows, heads * value_dim] in the compute type,
+    rows any stride."""
     _dev(raw, w, gate, out)
     rows = out.shape[0]
     ldh = value_dim + 2 if with_den else value_dim
     assert raw.dtype == torch.float32 and raw.is_contiguous() and raw.numel() == rows * heads * ldh
     assert w is None or (w.dtype == torch.float32 and w.numel() == (heads * value_dim if w_per_head else value_dim))
-    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and out.is_contiguous() and out.shape[1] == heads * value_dim
+    assert gate.dtype == torch.float32 and gate.stride(1) == 1 and out.stride(1) == 1 and out.shape[1] == heads * value_dim
     _check(_fn("recurrence", "cml_head_norm_gate")(_p(raw), ldh, 1 if with_den else 0, _p(w), value_dim if w_per_head else 0,
-                                                   _p(gate), gate.stride(0), gate_col, _p(out), dtype_code(out.dtype), rows,
-                                                   heads, value_dim, float(eps), 1 if gate_silu else 0, _stream()), "head_norm_gate")
+                                                   _p(gate), gate.stride(0), gate_col, _p(out), out.stride(0),
+                                                   dtype_code(out.dtype), rows, heads, value_dim, float(eps), 1 if gate_silu else 0, _stream()), "head_norm_gate")
+
+
+def delta_inputs(proj: torch.Tensor, a_bias: torch.Tensor, w0: torch.Tensor, rate: float, packed: torch.Tensor, scal: torch.Tensor,
+                 heads: int, key_dim: int, value_dim: int, high=None, w2=None, gate_out=None):
+    """What the generalized delta rule's scan reads, once per (row, head). ``proj`` (float32 [rows, n] or split sums
+    [splits, rows, n], added here): columns r, k (``heads`` x ``key_dim`` each), v (``heads`` x ``value_dim``), the removal
+    rates' inputs, the gate's (``heads`` x ``value_dim``), then the decays' narrow inputs. Rates a = sigmoid(in + ``a_bias``),
+    decays w = exp(-``rate`` sigmoid(z + ``w0``)) with z = ``high`` (float32 rows or split sums) or, without it, ``w2`` tanh(narrow
+    inputs), ``w2`` [heads * key_dim, rank]. ``packed`` [rows, heads, 4 key_dim + value_dim] and ``scal`` [rows, heads, 4], float32;
+    ``gate_out`` (float32 [rows, heads * value_dim]) gets the gate's summed inputs."""
+    _dev(proj, a_bias, w0, packed, scal, high, w2, gate_out)
+    if proj.dim() == 2:
+        proj = proj.unsqueeze(0)
+    if high is not None and high.dim() == 2:
+        high = high.unsqueeze(0)
+    rows, hd, hv = packed.shape[0], heads * key_dim, heads * value_dim
+    rank = w2.shape[1] if w2 is not None else 0
+    assert proj.dtype == torch.float32 and proj.stride(2) == 1 and proj.shape[1] == rows
+    assert proj.shape[2] >= 3 * hd + 2 * hv + (rank if high is None else 0)
+    assert packed.dtype == scal.dtype == torch.float32 and packed.is_contiguous() and scal.is_contiguous()
+    assert packed.shape == (rows, heads, 4 * key_dim + value_dim) and scal.shape == (rows, heads, 4)
+    assert a_bias.dtype == w0.dtype == torch.float32 and a_bias.numel() == hd == w0.numel()
+    assert high is None or (high.dtype == torch.float32 and high.shape[1:] == (rows, hd) and high.stride(2) == 1 and high.stride(1) == hd)
+    assert high is not None or (w2 is not None and w2.is_contiguous() and w2.shape[0] == hd)
+    assert gate_out is None or (gate_out.dtype == torch.float32 and gate_out.is_contiguous() and gate_out.shape == (rows, hv))
+    _check(_fn("recurrence", "cml_delta_inputs")(
+        _p(proj), proj.stride(1), proj.shape[0], proj.stride(0), _p(high), high.shape[0] if high is not None else 0,
+        high.stride(0) if high is not None else 0, _p(w2), dtype_code(w2.dtype) if w2 is not None else F32, rank, _p(a_bias), _p(w0),
+        float(rate), _p(packed), _p(scal), _p(gate_out), rows, heads, key_dim, value_dim, _stream()), "delta_inputs")
+
+
+def general_delta_scan(packed: torch.Tensor, scal: torch.Tensor, state: torch.Tensor, seq_row0, seq_new, seq_start, seq_slot,
+                       out: torch.Tensor, n_seqs: int, heads: int, key_dim: int, value_dim: int):
+    """The generalized delta rule over each sequence's new rows, S <- diag(w) S - (a * u)(u^T S) + k v^T, out = S^T r, on the
+    rows ``delta_inputs`` made; ``state`` float32 [slots, heads, value_dim, key_dim] (column by column) is read and replaced;
+    ``out`` float32 [rows, heads * value_dim]."""
+    _dev(packed, scal, state, seq_row0, seq_new, seq_start, seq_slot, out)
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (packed, scal, state, out))
+    assert packed.shape[1:] == (heads, 4 * key_dim + value_dim) and scal.shape[1:] == (heads, 4)
+    assert state.shape[1:] == (heads, value_dim, key_dim) and out.shape == (packed.shape[0], heads * value_dim)
+    _check(_fn("recurrence", "cml_general_delta_scan")(_p(packed), _p(scal), _p(state), _p(seq_row0), _p(seq_new), _p(seq_start),
+                                                       _p(seq_slot), _p(out), n_seqs, heads, key_dim, value_dim, _stream()),
+           "general_delta_scan")
 
 
 def rotate_rows_(x: torch.Tensor, col0: int, heads: int, head_dim: int, rotary_dim: int, interleaved: bool, inv_freq, amp: float,
@@ -839,29 +922,43 @@ def qkv_prepare(proj: torch.Tensor, q_w, k_w, norm_mode: int, eps: float, inv_fr
         float(amplitude), _stream()), "qkv_prepare")
 
 
-def latent_prepare(proj: torch.Tensor, c_w: torch.Tensor, eps: float, inv_freq, interleaved: bool, amplitude: float, row_seq,
-                   row_pos, table, q_plain, q_full, k_pages, heads: int, plain_dim: int, rot_dim: int, rank: int, extra_out=None):
+def latent_prepare(proj: torch.Tensor, c_w, eps: float, inv_freq, interleaved: bool, amplitude: float, row_seq,
+                   row_pos, table, q_plain, q_full, k_pages, heads: int, plain_dim: int, rot_dim: int, rank: int, extra_out=None,
+                   cq=None, cq_w=None):
     """The rows of a step for attention over a latent. ``proj`` (float32 [rows, n] or split sums [splits, rows, n], added
-    here) holds q (``heads`` x [``plain_dim`` unturned, ``rot_dim`` turned]), then ``rank`` + ``rot_dim`` columns of the down
-    projection, then the columns of ``extra_out`` (float32 [rows, e]). Writes the unturned query parts to ``q_plain``
-    [rows, heads * plain_dim], the turned ones to channels ``rank``.. of every head of ``q_full`` [rows, heads * (rank +
-    rot_dim)], and [rmsnorm(down[:rank]) * c_w, turned(down[rank:])] into the sequence's page row, all in the compute type."""
-    _dev(proj, c_w, inv_freq, row_seq, row_pos, table, q_plain, q_full, k_pages, extra_out)
-    rows = q_full.shape[0]
+    here) holds q (``heads`` x [``plain_dim`` unturned, ``rot_dim`` turned]; ``heads`` 0: none), then the columns of ``cq``
+    (a latent the queries are made from), then ``rank`` + ``rot_dim`` columns of the down projection (none where ``k_pages`` is
+    None), then the columns of ``extra_out`` (float32 [rows, e]). Writes the unturned query parts to ``q_plain`` [rows, heads *
+    plain_dim], the turned ones to channels ``rank``.. of every head of ``q_full`` [rows, heads * (rank + rot_dim)],
+    rmsnorm(query latent) * ``cq_w`` to ``cq`` [rows, n], and [rmsnorm(down[:rank]) * c_w, turned(down[rank:])] into the
+    sequence's page row, all in the compute type."""
+    _dev(proj, c_w, inv_freq, row_seq, row_pos, table, q_plain, q_full, k_pages, extra_out, cq, cq_w)
     if proj.dim() == 2:
         proj = proj.unsqueeze(0)
+    rows = proj.shape[1]
     extra = extra_out.shape[1] if extra_out is not None else 0
-    assert proj.dtype == torch.float32 and proj.stride(2) == 1 and proj.shape[1] == rows
-    assert proj.shape[2] >= heads * (plain_dim + rot_dim) + rank + rot_dim + extra
+    q_rank = cq.shape[1] if cq is not None else 0
+    down = k_pages is not None
+    assert proj.dtype == torch.float32 and proj.stride(2) == 1
+    assert proj.shape[2] >= heads * (plain_dim + rot_dim) + q_rank + (rank + rot_dim if down else 0) + extra
     assert extra_out is None or (extra_out.dtype == torch.float32 and extra_out.is_contiguous() and extra_out.shape[0] == rows)
-    assert q_plain.is_contiguous() and q_plain.shape == (rows, heads * plain_dim) and q_full.is_contiguous()
-    assert q_full.shape == (rows, heads * (rank + rot_dim)) and q_plain.dtype == q_full.dtype == k_pages.dtype
-    assert k_pages.is_contiguous() and k_pages.shape[1:] == (1, PAGE, rank + rot_dim) and c_w.numel() == rank
+    dtypes = {t.dtype for t in (q_plain, q_full, k_pages, cq) if t is not None}
+    assert len(dtypes) == 1
+    if heads:
+        assert q_plain.is_contiguous() and q_plain.shape == (rows, heads * plain_dim) and q_full.is_contiguous()
+        assert q_full.shape == (rows, heads * (rank + rot_dim))
+    w_dtypes = {t.dtype for t in (c_w if down else None, cq_w if q_rank else None) if t is not None}
+    assert len(w_dtypes) <= 1
+    if down:
+        assert k_pages.is_contiguous() and k_pages.shape[1:] == (1, PAGE, rank + rot_dim) and c_w.numel() == rank
+    if q_rank:
+        assert cq.is_contiguous() and cq.shape[0] == rows and cq_w.numel() == q_rank
     assert rot_dim == 0 or (inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dim // 2)
     _check(_fn("attention_latent", "cml_latent_prepare")(
-        _p(proj), proj.stride(1), proj.shape[0], proj.stride(0), extra, _p(extra_out), _p(c_w), dtype_code(c_w.dtype), float(eps),
-        _p(inv_freq), 1 if interleaved else 0, float(amplitude), _p(row_seq), _p(row_pos), _p(table), table.shape[1], _p(q_plain),
-        _p(q_full), _p(k_pages), dtype_code(q_full.dtype), rows, heads, plain_dim, rot_dim, rank, _stream()), "latent_prepare")
+        _p(proj), proj.stride(1), proj.shape[0], proj.stride(0), extra, _p(extra_out), _p(c_w), dtype_code(w_dtypes.pop() if w_dtypes else torch.float32),
+        float(eps), _p(inv_freq), 1 if interleaved else 0, float(amplitude), _p(row_seq), _p(row_pos), _p(table), table.shape[1],
+        _p(q_plain), _p(q_full), _p(k_pages), dtype_code(dtypes.pop()), rows, heads, plain_dim, rot_dim, rank, 1 if down else 0, q_rank,
+        _p(cq_w), _p(cq), _stream()), "latent_prepare")
 
 
 LATENT_PROMPT_ROWS = 64        # (token, head) query rows of a block of the prompt kernel; LA_ROWS in attention_latent.cu
@@ -881,13 +978,14 @@ def latent_prompt_usable(q: torch.Tensor, rank: int, rot_dim: int) -> bool:
 
 def latent_prompt(q_full, k_pages, out, table, tile_seq, tile_q0, n_tiles: int, seq_row0, seq_start, seq_new, heads: int,
                   rank: int, rot_dim: int, scale: float, sink=None, head_gate=None, gate_col: int = 0, partial=None,
-                  tiles_per_split: int = 0):
+                  tiles_per_split: int = 0, window: int = 0):
     """bfloat16 prompt attention over a latent on the tensor cores (mma.sync): ``q_full`` [rows, heads * (rank + rot_dim)]
-    against the sequences' cached rows [c, t] (``k_pages`` [pages, 1, 64, rank + rot_dim]), every earlier key visible;
+    against the sequences' cached rows [c, t] (``k_pages`` [pages, 1, 64, rank + rot_dim]), every earlier key visible or,
+    with ``window``, the row itself and the window - 1 before it;
     ``out`` [rows, heads * rank] gets the weighted latents per head, with exp(``sink``[head]) as one more term of the
     denominator and times sigmoid(``head_gate``[r, gate_col + head]). Tiles of ``latent_prompt_tokens(heads)`` tokens.
     ``partial`` (float32 [splits, rows, heads, rank + 2]; steps of one token per sequence only): a sequence's pages are
-    dealt to ``splits`` blocks, ``tiles_per_split`` pages each, and a second launch merges their shares in split order."""
+    dealt to ``splits`` blocks, ``tiles_per_split`` pages each (from the first page its window reaches on), and a second launch merges their shares in split order."""
     _dev(q_full, k_pages, out, table, tile_seq, tile_q0, seq_row0, seq_start, seq_new, sink, head_gate)
     rows, D = q_full.shape[0], rank + rot_dim
     assert latent_prompt_usable(q_full, rank, rot_dim) and q_full.is_contiguous() and q_full.shape[1] == heads * D
@@ -904,7 +1002,7 @@ def latent_prompt(q_full, k_pages, out, table, tile_seq, tile_q0, n_tiles: int, 
         _p(q_full), _p(k_pages), _p(out), _p(table), table.shape[1], _p(tile_seq), _p(tile_q0), int(n_tiles),
         1 if partial is not None else latent_prompt_tokens(heads), _p(seq_row0), _p(seq_start), _p(seq_new), _p(sink), _p(head_gate),
         head_gate.stride(0) if head_gate is not None else 0, int(gate_col), heads, rank, rot_dim, float(scale), _p(partial),
-        partial.shape[0] if partial is not None else 1, int(tiles_per_split), rows, _stream()),
+        partial.shape[0] if partial is not None else 1, int(tiles_per_split), rows, int(window), _stream()),
         "latent_prompt", 2 if partial is not None else 1)
 
 
@@ -925,22 +1023,24 @@ def head_product(x: torch.Tensor, x_head_stride: int, w: torch.Tensor, out: torc
 # routed feed-forwards
 
 def route_topk(logits: torch.Tensor, top: int, softmax: bool, renorm: bool, ids: torch.Tensor, wts: torch.Tensor,
-               correction=None, groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0):
+               correction=None, groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0, bias=None):
     """The ``top`` largest logits of every row: their expert ids and weights (sigmoid of the logit, or its softmax
     over all experts; ``renorm``: divided by the chosen weights' sum; times ``weight_scale``). logits float32 [rows,
     experts], or split sums [splits, rows, experts] that are added first. ``correction`` (float32 [experts]) is added
     to the scores for the choice only; with ``groups`` > 1 the experts form that many equal groups of neighbours and
-    only the ``keep_groups`` groups with the largest choice score of a member can be chosen from."""
-    _dev(logits, ids, wts, correction)
+    only the ``keep_groups`` groups with the largest choice score of a member can be chosen from. ``bias`` (float32
+    [experts]) is part of the logits."""
+    _dev(logits, ids, wts, correction, bias)
     assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous())
     if logits.dim() == 2:
         logits = logits.unsqueeze(0)
     _, rows, experts = logits.shape
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == experts)
     assert logits.dtype == torch.float32 and logits.stride(2) == 1 and ids.dtype == torch.int32 and wts.dtype == torch.float32
     assert ids.numel() == rows * top == wts.numel() and ids.is_contiguous() and wts.is_contiguous()
     _check(_fn("experts", "cml_route_topk")(_p(logits), logits.stride(1), logits.shape[0], logits.stride(0), rows, experts, int(top), 1 if softmax else 0,
                                             1 if renorm else 0, _p(correction), int(groups), int(keep_groups), float(weight_scale),
-                                            _p(ids), _p(wts), _stream()), "route_topk")
+                                            _p(ids), _p(wts), _p(bias), _stream()), "route_topk")
 
 
 EXPERT_TILE_ROWS, EXPERT_TILE_ROWS_TC = 64, 128      # rows of a tile of the grouped products: CUDA cores, tensor cores
@@ -1005,11 +1105,16 @@ def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogu
 
 
 def expert_combine(y: torch.Tensor, pos_of_pair, wts, top: int, scale_output: bool, shared, out: torch.Tensor,
-                   identity=None):
+                   identity=None, shared_gate=None, accumulate: bool = False):
     """out[row] = shared[row] + sum over the row's choices of y[place of the pair] (times its weight if
     ``scale_output``); ``shared`` float32 [rows, hidden] or [splits, rows, hidden] or None. ``identity`` = (ids,
     real_experts, rows): a choice of an expert ``real_experts`` or up adds ``rows[row]`` (float32 or bfloat16
-    [rows, hidden]) times its weight instead."""
+    [rows, hidden]) times its weight instead. ``shared_gate`` (float32 [rows, 1] or split sums [splits, rows, 1]): a logit
+    whose sigmoid multiplies the shared row. ``accumulate``: add to ``out`` instead of replacing it."""
+    if shared_gate is not None:
+        _dev(shared_gate)
+        shared_gate = shared_gate.unsqueeze(0) if shared_gate.dim() == 2 else shared_gate
+        assert shared_gate.dtype == torch.float32 and shared_gate.shape[1:] == (out.shape[0], 1)
     _dev(y, pos_of_pair, wts, shared, out)
     i_ids, i_real, i_rows = identity if identity is not None else (None, 0, None)
     if identity is not None:
@@ -1026,6 +1131,9 @@ def expert_combine(y: torch.Tensor, pos_of_pair, wts, top: int, scale_output: bo
     _check(_fn("experts", "cml_expert_combine")(_p(y), _p(pos_of_pair), _p(wts), int(top), 1 if scale_output else 0, _p(shared),
                                                 splits, stride, _p(i_ids), int(i_real), _p(i_rows),
                                                 dtype_code(i_rows.dtype) if i_rows is not None else 0, _p(out), rows, hidden,
+                                                _p(shared_gate), shared_gate.stride(1) if shared_gate is not None else 0,
+                                                shared_gate.shape[0] if shared_gate is not None else 0,
+                                                shared_gate.stride(0) if shared_gate is not None else 0, 1 if accumulate else 0,
                                                 _stream()), "expert_combine")
 
 

@@ -8,6 +8,8 @@
 //                                                  o = S^T q / (max(|n . q|, e^(-m')) + 1e-6)
 //
 //   retention (a fixed decay per head):            S <- d S + k v^T;  o = S^T q
+//   generalized delta rule (decay w and removal rate a per key channel, u = k / |k|):
+//                                                  S <- diag(w) S - (a * u)(u^T S) + k v^T;  o = S^T r
 //
 // All are independent per column of S: eight threads of a warp share one column (a slice of
 // the key axis each, in registers) of one (sequence, head) and walk the sequence's new tokens
@@ -499,6 +501,287 @@ extern "C" int cml_retention_scan(const float* proj, long ld, int q_col, int k_c
 }
 
 // ------------------------------------------------------------------------------------
+// Generalized delta rule. Both terms of the write read the old state, so with p = k^T S (S before the token), q = (r * w)^T S,
+// n2 = 1 / (sum k^2 + 1e-6) the token is
+//
+//   S' = diag(w) S + k (v - a * (n2 p))^T,     o = q - n2 (sum r a k) p + (sum r k) v
+//
+// and the two products over the state, p and q, are taken side by side. What does not depend on the state is made
+// beforehand, once per (row, head), by the kernel below: `packed` [rows, heads, 4 D + Dv] = k, r * w, w, a, v and `scal`
+// [rows, heads, 4] = n2, n2 sum r a k, sum r k, 0.
+//
+// proj (n_splits matrices split_stride apart, added in split order) [rows, ld]: columns r, k (heads x D each), v
+// (heads x Dv), the removal rates' inputs (heads x D), the gate's (heads x Dv), then `rank` columns of the decays' narrow
+// inputs. a = sigmoid(in + a_bias). The decays' inputs z come as a product of their own (`high`, n_high matrices
+// high_stride apart [rows, heads x D]) or, where `high` is null, are made here: z = W2 tanh(narrow), W2 [heads x D, rank].
+// w = exp(-rate * sigmoid(z + w0)). gate_out (may be null) gets the gate's summed inputs [rows, heads x Dv].
+struct DeltaInputs {
+    const float* proj; long ld; int n_splits; long split_stride;
+    const float* high; int n_high; long high_stride;
+    const void* w2; int rank;
+    const float* a_bias; const float* w0;
+    float rate;
+    float* packed; float* scal; float* gate_out;
+    int heads, D, Dv;
+};
+
+__device__ __forceinline__ float split_sum(const float* p, int n, long stride) {
+    float v = p[0];
+    for (int s0 = 1; s0 < n; s0 += 8) {                        // eight splits' loads in flight, added in split order
+        float t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = p[(size_t)min(s0 + k, n - 1) * stride];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += s0 + k < n ? t[k] : 0.f;
+    }
+    return v;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_inputs_kernel(const DeltaInputs p) {
+    extern __shared__ __align__(16) float di_low[];            // tanh of the narrow inputs
+    __shared__ float red0[32], red1[32], red2[32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = blockIdx.x, hd = blockIdx.y, D = p.D, Dv = p.Dv, HD = p.heads * p.D, HV = p.heads * p.Dv;
+    const float* row = p.proj + (size_t)r * p.ld;
+    if (p.high == nullptr) {
+        const float* narrow = row + 3 * HD + 2 * HV;
+        for (int j = threadIdx.x; j < p.rank; j += blockDim.x) di_low[j] = tanhf(split_sum(narrow + j, p.n_splits, p.split_stride));
+        __syncthreads();
+    }
+    float* pk = p.packed + ((size_t)r * p.heads + hd) * (4 * D + Dv);
+    float k2 = 0.f, rak = 0.f, rk = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+        const int c = hd * D + d;
+        const float rr = split_sum(row + c, p.n_splits, p.split_stride);
+        const float kk = split_sum(row + HD + c, p.n_splits, p.split_stride);
+        const float aa = sigmoid_f(split_sum(row + 2 * HD + HV + c, p.n_splits, p.split_stride) + p.a_bias[c]);
+        float z = 0.f;
+        if (p.high != nullptr) {
+            z = split_sum(p.high + (size_t)r * HD + c, p.n_high, p.high_stride);
+        } else {
+            const T* w = (const T*)p.w2 + (size_t)c * p.rank;
+            constexpr int PIECE = 16 / (int)sizeof(T);
+            int j = 0;
+            if (p.rank % PIECE == 0 && (((uintptr_t)p.w2) & 15) == 0) {
+                for (; j < p.rank; j += PIECE) {
+                    union { uint4 raw; T e[PIECE]; } v;
+                    v.raw = *reinterpret_cast<const uint4*>(w + j);
+#pragma unroll
+                    for (int e = 0; e < PIECE; ++e) z = fmaf(to_f32(v.e[e]), di_low[j + e], z);
+                }
+            } else {
+                for (; j < p.rank; ++j) z = fmaf(to_f32(w[j]), di_low[j], z);
+            }
+        }
+        const float ww = expf(-p.rate * sigmoid_f(z + p.w0[c]));
+        pk[d] = kk;
+        pk[D + d] = rr * ww;
+        pk[2 * D + d] = ww;
+        pk[3 * D + d] = aa;
+        k2 = fmaf(kk, kk, k2);
+        rak = fmaf(rr * aa, kk, rak);
+        rk = fmaf(rr, kk, rk);
+    }
+    for (int c = threadIdx.x; c < Dv; c += blockDim.x) {
+        pk[4 * D + c] = split_sum(row + 2 * HD + hd * Dv + c, p.n_splits, p.split_stride);
+        if (p.gate_out) p.gate_out[(size_t)r * HV + hd * Dv + c] = split_sum(row + 3 * HD + HV + hd * Dv + c, p.n_splits, p.split_stride);
+    }
+    k2 = block_sum(k2, red0);
+    rak = block_sum(rak, red1);
+    rk = block_sum(rk, red2);
+    if (threadIdx.x == 0) {
+        const float n2 = 1.0f / (k2 + 1e-6f);
+        float4* out = reinterpret_cast<float4*>(p.scal + ((size_t)r * p.heads + hd) * 4);
+        *out = make_float4(n2, n2 * rak, rk, 0.f);
+    }
+}
+
+extern "C" int cml_delta_inputs(const float* proj, long ld, int n_splits, long split_stride, const float* high, int n_high,
+                                long high_stride, const void* w2, int dtype, int rank, const float* a_bias, const float* w0,
+                                float rate, float* packed, float* scal, float* gate_out, int rows, int heads, int D, int Dv,
+                                void* stream) {
+    if (rows <= 0) return 0;
+    if (heads < 1 || heads > 65535 || D < 1 || Dv < 1 || n_splits < 1 || rank < 0 || rank > 8192) return CML_ERR_BAD_SIZE;
+    if (high == nullptr ? w2 == nullptr : n_high < 1) return CML_ERR_BAD_SIZE;
+    if (((uintptr_t)scal) & 15) return CML_ERR_BAD_ALIGN;
+    DeltaInputs p = {proj, ld, n_splits, split_stride, high, n_high, high_stride, w2, rank, a_bias, w0, rate, packed, scal, gate_out,
+                     heads, D, Dv};
+    const int most = D > Dv ? D : Dv;
+    const int block = most >= 256 ? 256 : (most + 31) / 32 * 32;
+    const size_t smem = high == nullptr ? (size_t)rank * sizeof(float) : 0;
+    if (dtype == CML_DTYPE_F32)
+        launch_pdl(delta_inputs_kernel<float>, dim3(rows, heads), dim3(block), smem, (cudaStream_t)stream, p);
+    else if (dtype == CML_DTYPE_BF16)
+        launch_pdl(delta_inputs_kernel<bf16>, dim3(rows, heads), dim3(block), smem, (cudaStream_t)stream, p);
+    else
+        return CML_ERR_BAD_DTYPE;
+    return cml_launch_status();
+}
+
+// The scan: like the scans above a block of 128 threads owns 128 / NS columns of one (sequence, head), NS threads of a warp
+// share a column (a slice of DS key channels each) and walk the new tokens in order. The prepared rows of
+// GD_TOKENS tokens come by cp.async into one of two buffers of shared memory while the other one's are worked on.
+#define GD_TOKENS 8
+struct GeneralDelta {
+    const float* packed; const float* scal; float* state;
+    const int* seq_row0; const int* seq_new; const int* seq_start; const int* seq_slot;
+    float* out;
+    int heads, D, Dv;
+};
+
+template <int BYTES>
+__device__ __forceinline__ void gd_copy(float* smem, const float* gmem) {
+    const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
+    if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(s), "l"(gmem) : "memory");
+}
+
+template <int DS, int NS>
+__global__ void __launch_bounds__(128) general_delta_kernel(const GeneralDelta p) {
+    constexpr int COLS = 128 / NS;
+    constexpr int SL = DS == 4 ? 4 : DS + 4;               // floats of a slice in shared memory (padded against bank conflicts)
+    constexpr int ROW = NS * SL;                           // floats of one array of a token
+    constexpr int TOKEN = 4 * ROW + COLS + 4;              // k, r * w, w, a; the block's values; the scalars
+    extern __shared__ __align__(16) float gd_sh[];         // [2][GD_TOKENS][TOKEN]
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, hd = blockIdx.y;
+    const int D = p.D, Dv = p.Dv, heads = p.heads;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, slice = lane % NS;
+    const int wcol = warp * (32 / NS) + lane / NS;
+    const int col0 = blockIdx.z * COLS, c = col0 + wcol;
+    const bool live = c < Dv;
+    const int d0 = slice * DS;
+    const int row0 = p.seq_row0[s], n = p.seq_new[s];
+    const bool fresh = p.seq_start[s] == 0, vec = ((D | Dv) & 3) == 0;     // whole heads of `packed` start on 16 bytes
+    const size_t per_head = 4 * D + Dv, per_row = per_head * heads;
+    float* st = p.state + (((size_t)p.seq_slot[s] * heads + hd) * Dv + (live ? c : 0)) * D;
+    auto fetch = [&](int t0, int buf) {
+        const int nt = min(GD_TOKENS, n - t0);
+        float* dst = gd_sh + (size_t)buf * GD_TOKENS * TOKEN;
+        const float* src = p.packed + (size_t)(row0 + t0) * per_row + (size_t)hd * per_head;
+        if (vec) {
+            const int q = D / 4;                           // 16-byte pieces of an array; a warp takes every fourth (token, array)
+            for (int ta = warp; ta < 4 * nt; ta += 4)
+                for (int i = lane; i < q; i += 32) {
+                    const int d = 4 * i;
+                    gd_copy<16>(dst + (ta >> 2) * TOKEN + (ta & 3) * ROW + (d / DS) * SL + d % DS, src + (size_t)(ta >> 2) * per_row + (ta & 3) * D + d);
+                }
+        } else {
+            for (int ta = warp; ta < 4 * nt; ta += 4)
+                for (int d = lane; d < D; d += 32)
+                    gd_copy<4>(dst + (ta >> 2) * TOKEN + (ta & 3) * ROW + (d / DS) * SL + d % DS, src + (size_t)(ta >> 2) * per_row + (ta & 3) * D + d);
+        }
+        for (int i = threadIdx.x; i < nt * COLS; i += 128) {
+            const int t = i / COLS, cc = i % COLS;
+            if (col0 + cc < Dv) gd_copy<4>(dst + t * TOKEN + 4 * ROW + cc, src + (size_t)t * per_row + 4 * D + col0 + cc);
+        }
+        if (threadIdx.x < nt)
+            gd_copy<16>(dst + threadIdx.x * TOKEN + 4 * ROW + COLS, p.scal + ((size_t)(row0 + t0 + threadIdx.x) * heads + hd) * 4);
+    };
+    if (D < NS * DS || Dv - col0 < COLS) {                 // channels and columns that are not there stay zero
+        for (int i = threadIdx.x; i < 2 * GD_TOKENS * TOKEN; i += 128) gd_sh[i] = 0.f;
+        __syncthreads();
+    }
+    fetch(0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    float S[DS];
+#pragma unroll
+    for (int i = 0; i < DS; i += 4) {
+        if (live && !fresh && vec && d0 + i < D) {
+            const float4 t = *reinterpret_cast<const float4*>(st + d0 + i);
+            S[i] = t.x; S[i + 1] = t.y; S[i + 2] = t.z; S[i + 3] = t.w;
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) S[i + j] = (live && !fresh && d0 + i + j < D) ? st[d0 + i + j] : 0.f;
+        }
+    }
+    for (int t0 = 0, buf = 0; t0 < n; t0 += GD_TOKENS, buf ^= 1) {
+        if (t0 + GD_TOKENS < n) fetch(t0 + GD_TOKENS, buf ^ 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");           // all but the newest group: this round's tokens are here
+        __syncthreads();
+        const float* base = gd_sh + (size_t)buf * GD_TOKENS * TOKEN;
+        auto token = [&](int t) {
+            const float* tk = base + t * TOKEN + slice * SL;
+            const float vcol = base[t * TOKEN + 4 * ROW + wcol];
+            const float4 sc = *reinterpret_cast<const float4*>(base + t * TOKEN + 4 * ROW + COLS);
+            float kr[DS], p4[4] = {0.f, 0.f, 0.f, 0.f}, q4[4] = {0.f, 0.f, 0.f, 0.f};      // four chains each, always in this order
+#pragma unroll
+            for (int i = 0; i < DS; i += 4) {
+                const float4 kv = *reinterpret_cast<const float4*>(tk + i), rv = *reinterpret_cast<const float4*>(tk + ROW + i);
+                kr[i] = kv.x; kr[i + 1] = kv.y; kr[i + 2] = kv.z; kr[i + 3] = kv.w;
+                p4[0] = fmaf(S[i], kv.x, p4[0]); p4[1] = fmaf(S[i + 1], kv.y, p4[1]);
+                p4[2] = fmaf(S[i + 2], kv.z, p4[2]); p4[3] = fmaf(S[i + 3], kv.w, p4[3]);
+                q4[0] = fmaf(S[i], rv.x, q4[0]); q4[1] = fmaf(S[i + 1], rv.y, q4[1]);
+                q4[2] = fmaf(S[i + 2], rv.z, q4[2]); q4[3] = fmaf(S[i + 3], rv.w, q4[3]);
+            }
+            float pk = (p4[0] + p4[1]) + (p4[2] + p4[3]), qr = (q4[0] + q4[1]) + (q4[2] + q4[3]);
+#pragma unroll
+            for (int sh = 1; sh < NS; sh <<= 1) {
+                const float x = __shfl_xor_sync(0xffffffffu, pk, sh), y = __shfl_xor_sync(0xffffffffu, qr, sh);
+                pk += x;
+                qr += y;
+            }
+            const float rem = -sc.x * pk;
+#pragma unroll
+            for (int i = 0; i < DS; i += 4) {
+                const float4 wv = *reinterpret_cast<const float4*>(tk + 2 * ROW + i), av = *reinterpret_cast<const float4*>(tk + 3 * ROW + i);
+                S[i] = fmaf(kr[i], fmaf(av.x, rem, vcol), wv.x * S[i]);
+                S[i + 1] = fmaf(kr[i + 1], fmaf(av.y, rem, vcol), wv.y * S[i + 1]);
+                S[i + 2] = fmaf(kr[i + 2], fmaf(av.z, rem, vcol), wv.z * S[i + 2]);
+                S[i + 3] = fmaf(kr[i + 3], fmaf(av.w, rem, vcol), wv.w * S[i + 3]);
+            }
+            if (live && slice == 0)
+                p.out[((size_t)(row0 + t0 + t) * heads + hd) * Dv + c] = fmaf(sc.z, vcol, fmaf(-sc.y, pk, qr));
+        };
+        const int nt = min(GD_TOKENS, n - t0);
+        if (nt == GD_TOKENS) {                             // a whole round unrolled: the next tokens' loads and this one's read-out overlap
+#pragma unroll
+            for (int t = 0; t < GD_TOKENS; ++t) token(t);
+        } else {
+            for (int t = 0; t < nt; ++t) token(t);
+        }
+        __syncthreads();                                   // before the next fetch overwrites this buffer
+    }
+    if (live) {
+#pragma unroll
+        for (int i = 0; i < DS; i += 4) {
+            if (vec && d0 + i < D) {
+                *reinterpret_cast<float4*>(st + d0 + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (d0 + i + j < D) st[d0 + i + j] = S[i + j];
+            }
+        }
+    }
+}
+
+extern "C" int cml_general_delta_scan(const float* packed, const float* scal, float* state, const int* seq_row0, const int* seq_new,
+                                      const int* seq_start, const int* seq_slot, float* out, int n_seqs, int heads, int D, int Dv,
+                                      void* stream) {
+    if (n_seqs <= 0) return 0;
+    if (D < 1 || D > 256 || Dv < 1 || heads < 1 || heads > 65535) return CML_ERR_BAD_SIZE;
+    if ((((uintptr_t)packed) | ((uintptr_t)scal) | ((uintptr_t)state)) & 15) return CML_ERR_BAD_ALIGN;
+    GeneralDelta p = {packed, scal, state, seq_row0, seq_new, seq_start, seq_slot, out, heads, D, Dv};
+    constexpr int NS = SCAN_SLICES, COLS = 128 / NS;
+    dim3 grid(n_seqs, heads, (Dv + COLS - 1) / COLS);
+#define GD_CASE(DS_)                                                                                                     \
+    if (D <= NS * DS_) {                                                                                                 \
+        constexpr size_t smem = (size_t)2 * GD_TOKENS * (4 * NS * (DS_ == 4 ? 4 : DS_ + 4) + COLS + 4) * sizeof(float);  \
+        if (smem > 48 * 1024 && cml_allow_smem<general_delta_kernel<DS_, NS>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE; \
+        launch_pdl(general_delta_kernel<DS_, NS>, grid, dim3(128), smem, (cudaStream_t)stream, p);                       \
+        return cml_launch_status();                                                                                      \
+    }
+    GD_CASE(4) GD_CASE(8) GD_CASE(16) GD_CASE(32)
+#undef GD_CASE
+    return CML_ERR_BAD_SIZE;
+}
+
+// ------------------------------------------------------------------------------------
 // Rotation of heads inside float rows, in place: x [rows, ld] holds `heads` heads of D channels from column col0; the
 // first rot_dim channels of every head are turned by angle = position * inv_freq[i] (pairing 1: channels (2i, 2i + 1);
 // 0: channels (i, i + rot_dim / 2)), sines and cosines times `amp`; then heads from number `scaled_from` on are
@@ -548,7 +831,7 @@ extern "C" int cml_rotate_rows(float* x, long ld, int col0, int rows, int heads,
 template <typename TO>
 __global__ void head_norm_gate_kernel(const float* __restrict__ raw, int ldh, int with_den, const float* __restrict__ w,
                                       int w_head_stride, const float* __restrict__ gate, long ldg, int gate_col,
-                                      TO* __restrict__ out, int rows, int heads, int Dv, float eps, int gate_silu) {
+                                      TO* __restrict__ out, long ldo, int rows, int heads, int Dv, float eps, int gate_silu) {
     pdl_wait();
     pdl_launch_dependents();
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -566,12 +849,12 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ raw, int ldh, in
     const float scale = inv / sqrtf(ss / (float)Dv + eps);
     const float* wv = w ? w + (size_t)hd * w_head_stride : nullptr;      // null: a norm without weight
     const float* gt = gate + (size_t)r * ldg + gate_col + hd * Dv;
-    TO* o = out + ((size_t)r * heads + hd) * Dv;
+    TO* o = out + (size_t)r * ldo + (size_t)hd * Dv;
     for (int c = lane; c < Dv; c += 32) o[c] = from_f32<TO>(x[c] * scale * (wv ? wv[c] : 1.0f) * (gate_silu ? silu_f(gt[c]) : sigmoid_f(gt[c])));
 }
 
 extern "C" int cml_head_norm_gate(const float* raw, int ldh, int with_den, const float* w, int w_head_stride, const float* gate,
-                                  long ldg, int gate_col, void* out, int out_dtype, int rows, int heads, int Dv, float eps,
+                                  long ldg, int gate_col, void* out, long ldo, int out_dtype, int rows, int heads, int Dv, float eps,
                                   int gate_silu, void* stream) {
     if (rows <= 0) return 0;
     const long warps = (long)rows * heads;
@@ -579,10 +862,10 @@ extern "C" int cml_head_norm_gate(const float* raw, int ldh, int with_den, const
     cudaStream_t s = (cudaStream_t)stream;
     if (out_dtype == CML_DTYPE_F32)
         launch_pdl(head_norm_gate_kernel<float>, grid, dim3(128), 0, s, raw, ldh, with_den, w, w_head_stride, gate, ldg, gate_col,
-                   (float*)out, rows, heads, Dv, eps, gate_silu);
+                   (float*)out, ldo, rows, heads, Dv, eps, gate_silu);
     else if (out_dtype == CML_DTYPE_BF16)
         launch_pdl(head_norm_gate_kernel<bf16>, grid, dim3(128), 0, s, raw, ldh, with_den, w, w_head_stride, gate, ldg, gate_col,
-                   (bf16*)out, rows, heads, Dv, eps, gate_silu);
+                   (bf16*)out, ldo, rows, heads, Dv, eps, gate_silu);
     else
         return CML_ERR_BAD_DTYPE;
     return cml_launch_status();

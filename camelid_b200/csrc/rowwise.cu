@@ -99,10 +99,12 @@ extern "C" int cml_embed_positions(const void* table, int dtype, const int* toke
 // `partial` (may be null) holds `n_splits` float matrices [x_rows, hidden] that are still to
 // be added to x (the split sums of the product before): they are added in index order, and
 // without `rows_index` the sum is written back to x, which settles the residual stream.
+// `w2` / `out2` (may be null): a second norm of the same rows that differs in its weight alone, out of the same pass.
 template <typename TW, typename TO>
 __global__ void rmsnorm_kernel(float* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out,
                                const int* __restrict__ rows_index, int hidden, float eps,
-                               const float* __restrict__ partial, int n_splits, size_t split_stride) {
+                               const float* __restrict__ partial, int n_splits, size_t split_stride,
+                               const TW* __restrict__ w2, TO* __restrict__ out2) {
     __shared__ float red[33];
     extern __shared__ float rowbuf[];
     // the norm's weight does not depend on the kernels before: its first columns are fetched
@@ -160,6 +162,7 @@ __global__ void rmsnorm_kernel(float* __restrict__ x, const TW* __restrict__ w, 
         const float v = partial ? rowbuf[c] : xr[c];
         const float wc = c == c0 ? w0 : (c == c1 ? w1 : to_f32(w[c]));
         o[c] = from_f32<TO>(v * scale * wc);
+        if (w2) out2[(size_t)r * hidden + c] = from_f32<TO>(v * scale * to_f32(w2[c]));
     }
 }
 
@@ -173,7 +176,7 @@ template <typename TW, typename TO>
 __global__ void rmsnorm_settle_kernel(float* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out,
                                       const int* __restrict__ rows_index, int hidden, float eps,
                                       const float* __restrict__ partial, int n_splits, size_t split_stride,
-                                      int units_per_round) {
+                                      int units_per_round, const TW* __restrict__ w2, TO* __restrict__ out2) {
     __shared__ float red[33];
     extern __shared__ __align__(16) float dyn[];
     float4* rowbuf = reinterpret_cast<float4*>(dyn);
@@ -182,9 +185,14 @@ __global__ void rmsnorm_settle_kernel(float* __restrict__ x, const TW* __restric
     const int groups = hidden >> 2;
     const int g0 = threadIdx.x;
     float wv[4] = {0.f, 0.f, 0.f, 0.f};             // the norm's weight does not depend on the kernels before
+    float wv2[4] = {0.f, 0.f, 0.f, 0.f};
     if (g0 < groups) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) wv[i] = to_f32(w[4 * g0 + i]);
+        if (w2) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) wv2[i] = to_f32(w2[4 * g0 + i]);
+        }
     }
     const int r = blockIdx.x;
     const int units = n_splits + 1;                 // unit 0: the row itself; unit u: split u - 1
@@ -233,12 +241,21 @@ __global__ void rmsnorm_settle_kernel(float* __restrict__ x, const TW* __restric
         o[4 * g + 1] = from_f32<TO>(v.y * scale * wc[1]);
         o[4 * g + 2] = from_f32<TO>(v.z * scale * wc[2]);
         o[4 * g + 3] = from_f32<TO>(v.w * scale * wc[3]);
+        if (w2) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) wc[i] = g == g0 ? wv2[i] : to_f32(w2[4 * g + i]);
+            TO* o2 = out2 + (size_t)r * hidden + 4 * g;
+            o2[0] = from_f32<TO>(v.x * scale * wc[0]);
+            o2[1] = from_f32<TO>(v.y * scale * wc[1]);
+            o2[2] = from_f32<TO>(v.z * scale * wc[2]);
+            o2[3] = from_f32<TO>(v.w * scale * wc[3]);
+        }
     }
 }
 
 template <typename TW, typename TO>
 static int launch_rmsnorm_settle(float* x, const void* w, void* out, const int* rows_index, int rows, int hidden, float eps,
-                                 const float* partial, int n_splits, long split_stride, cudaStream_t s) {
+                                 const float* partial, int n_splits, long split_stride, const void* w2, void* out2, cudaStream_t s) {
     const int groups = hidden / 4;
     int block = ((groups + 31) / 32) * 32;
     if (block > 1024) block = 1024;
@@ -250,7 +267,7 @@ static int launch_rmsnorm_settle(float* x, const void* w, void* out, const int* 
     cudaError_t e = cml_allow_smem<rmsnorm_settle_kernel<TW, TO>>(smem);
     if (e != cudaSuccess) return (int)e;
     launch_pdl(rmsnorm_settle_kernel<TW, TO>, dim3(rows), dim3(block), smem, s, x, (const TW*)w, (TO*)out, rows_index, hidden,
-               eps, partial, n_splits, (size_t)split_stride, upr);
+               eps, partial, n_splits, (size_t)split_stride, upr, (const TW*)w2, (TO*)out2);
     return cml_launch_status();
 }
 
@@ -259,7 +276,8 @@ static int launch_rmsnorm_settle(float* x, const void* w, void* out, const int* 
 template <typename TW, typename TO, int VPL>
 __global__ void __launch_bounds__(256)
 rmsnorm_rows_kernel(const float* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out,
-                    const int* __restrict__ rows_index, int rows, int hidden, float eps) {
+                    const int* __restrict__ rows_index, int rows, int hidden, float eps, const TW* __restrict__ w2,
+                    TO* __restrict__ out2) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -283,25 +301,28 @@ rmsnorm_rows_kernel(const float* __restrict__ x, const TW* __restrict__ w, TO* _
     }
     ss = warp_sum(ss);
     const float scale = 1.0f / sqrtf(ss / (float)hidden + eps);
-    TO* o = out + (size_t)r * hidden;
+    auto write = [&](const TW* wt, TO* o) {
 #pragma unroll
-    for (int i = 0; i < VPL; ++i) {
-        const int c = (lane + 32 * i) * 4;
-        if (c >= hidden) continue;
-        o[c] = from_f32<TO>(v[i].x * scale * to_f32(w[c]));
-        o[c + 1] = from_f32<TO>(v[i].y * scale * to_f32(w[c + 1]));
-        o[c + 2] = from_f32<TO>(v[i].z * scale * to_f32(w[c + 2]));
-        o[c + 3] = from_f32<TO>(v[i].w * scale * to_f32(w[c + 3]));
-    }
+        for (int i = 0; i < VPL; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            if (c >= hidden) continue;
+            o[c] = from_f32<TO>(v[i].x * scale * to_f32(wt[c]));
+            o[c + 1] = from_f32<TO>(v[i].y * scale * to_f32(wt[c + 1]));
+            o[c + 2] = from_f32<TO>(v[i].z * scale * to_f32(wt[c + 2]));
+            o[c + 3] = from_f32<TO>(v[i].w * scale * to_f32(wt[c + 3]));
+        }
+    };
+    write(w, out + (size_t)r * hidden);
+    if (w2) write(w2, out2 + (size_t)r * hidden);
 }
 
 template <typename TW, typename TO>
 static bool launch_rmsnorm_rows(const float* x, const void* w, void* out, const int* rows_index, int rows, int hidden,
-                                float eps, cudaStream_t s) {
+                                float eps, const void* w2, void* out2, cudaStream_t s) {
     if (hidden % 4 != 0 || hidden > 4096 || rows < 64) return false;
     const dim3 grid((rows + 7) / 8), block(256);
     const int vpl = (hidden / 4 + 31) / 32;
-#define CML_ROWS(V) launch_pdl(rmsnorm_rows_kernel<TW, TO, V>, grid, block, 0, s, x, (const TW*)w, (TO*)out, rows_index, rows, hidden, eps)
+#define CML_ROWS(V) launch_pdl(rmsnorm_rows_kernel<TW, TO, V>, grid, block, 0, s, x, (const TW*)w, (TO*)out, rows_index, rows, hidden, eps, (const TW*)w2, (TO*)out2)
     if (vpl <= 4) CML_ROWS(4);
     else if (vpl <= 8) CML_ROWS(8);
     else if (vpl <= 16) CML_ROWS(16);
@@ -313,30 +334,31 @@ static bool launch_rmsnorm_rows(const float* x, const void* w, void* out, const 
 
 extern "C" int cml_rmsnorm(float* x, const void* w, int w_dtype, void* out, int out_dtype,
                            const int* rows_index, int rows, int hidden, float eps, const float* partial,
-                           int n_splits, long split_stride, void* stream) {
+                           int n_splits, long split_stride, const void* w2, void* out2, void* stream) {
     if (rows <= 0) return 0;
+    if (w2 != nullptr && out2 == nullptr) return CML_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     if (!partial) {
         bool done = false;
-        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_F32) done = launch_rmsnorm_rows<float, float>(x, w, out, rows_index, rows, hidden, eps, s);
-        else if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_BF16) done = launch_rmsnorm_rows<float, bf16>(x, w, out, rows_index, rows, hidden, eps, s);
-        else if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_F32) done = launch_rmsnorm_rows<bf16, float>(x, w, out, rows_index, rows, hidden, eps, s);
-        else if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_BF16) done = launch_rmsnorm_rows<bf16, bf16>(x, w, out, rows_index, rows, hidden, eps, s);
+        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_F32) done = launch_rmsnorm_rows<float, float>(x, w, out, rows_index, rows, hidden, eps, w2, out2, s);
+        else if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_BF16) done = launch_rmsnorm_rows<float, bf16>(x, w, out, rows_index, rows, hidden, eps, w2, out2, s);
+        else if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_F32) done = launch_rmsnorm_rows<bf16, float>(x, w, out, rows_index, rows, hidden, eps, w2, out2, s);
+        else if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_BF16) done = launch_rmsnorm_rows<bf16, bf16>(x, w, out, rows_index, rows, hidden, eps, w2, out2, s);
         if (done) return cml_launch_status();
     }
     if (partial && hidden % 4 == 0 && split_stride % 4 == 0 && (((uintptr_t)x | (uintptr_t)partial) & 15) == 0 &&
         (size_t)hidden * sizeof(float) <= 100 * 1024) {
-        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_F32) return launch_rmsnorm_settle<float, float>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, s);
-        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_BF16) return launch_rmsnorm_settle<float, bf16>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, s);
-        if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_F32) return launch_rmsnorm_settle<bf16, float>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, s);
-        if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_BF16) return launch_rmsnorm_settle<bf16, bf16>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, s);
+        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_F32) return launch_rmsnorm_settle<float, float>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, w2, out2, s);
+        if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_BF16) return launch_rmsnorm_settle<float, bf16>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, w2, out2, s);
+        if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_F32) return launch_rmsnorm_settle<bf16, float>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, w2, out2, s);
+        if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_BF16) return launch_rmsnorm_settle<bf16, bf16>(x, w, out, rows_index, rows, hidden, eps, partial, n_splits, split_stride, w2, out2, s);
         return CML_ERR_BAD_DTYPE;
     }
     // few rows (decode): many threads per row shorten the chain; many rows: several blocks per SM
     const int block = hidden >= 1024 ? (rows <= 256 ? 1024 : 256) : (hidden >= 512 ? 256 : 128);
     const size_t smem = partial ? (size_t)hidden * sizeof(float) : 0;
     if (smem > 48 * 1024) return CML_ERR_BAD_SIZE;
-#define CML_RMS(TW, TO) launch_pdl(rmsnorm_kernel<TW, TO>, dim3(rows), dim3(block), smem, s, x, (const TW*)w, (TO*)out, rows_index, hidden, eps, partial, n_splits, (size_t)split_stride)
+#define CML_RMS(TW, TO) launch_pdl(rmsnorm_kernel<TW, TO>, dim3(rows), dim3(block), smem, s, x, (const TW*)w, (TO*)out, rows_index, hidden, eps, partial, n_splits, (size_t)split_stride, (const TW*)w2, (TO*)out2)
     if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_F32) CML_RMS(float, float);
     else if (w_dtype == CML_DTYPE_F32 && out_dtype == CML_DTYPE_BF16) CML_RMS(float, bf16);
     else if (w_dtype == CML_DTYPE_BF16 && out_dtype == CML_DTYPE_F32) CML_RMS(bf16, float);

@@ -397,6 +397,137 @@ extern "C" int cml_act_from_partials(const float* part, int n_splits, long strid
     return cml_launch_status();
 }
 
+// out[r] = a N(z) + b N(z^2) + c N(z^3) + e of a row z of `width` values, powers taken element by element, N(y) = y /
+// sqrt(mean(y^2) + eps); (a, b, c, e) = coef[0..3] on the device. z comes as float split sums (n_splits matrices
+// split_stride apart, rows ldz apart) that are added in split order, or as rows of the compute type (part null), which
+// may be the output's own. One block per row; the row stays in shared memory between the two passes; sums in float.
+template <typename T>
+__global__ void __launch_bounds__(512) poly_norm_kernel(const float* __restrict__ part, int n_splits, long split_stride, long ldz,
+                                                        const T* z_rows, const float* __restrict__ coef, float eps, T* out, long ldo,
+                                                        int width) {
+    extern __shared__ __align__(16) float pn_row[];
+    __shared__ float red0[32], red1[32], red2[32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = blockIdx.x;
+    float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+    auto count = [&](float v) {
+        const float q = v * v, q2 = q * q;
+        s2 += q;
+        s4 += q2;
+        s6 = fmaf(q2, q, s6);
+    };
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const bool vec = width % VEC == 0 && ldo % VEC == 0 && ((uintptr_t)out & 15) == 0 &&
+                     (part ? (((uintptr_t)part & 15) == 0 && split_stride % 4 == 0 && ldz % 4 == 0)
+                           : (((uintptr_t)z_rows & 15) == 0 && ldz % VEC == 0));
+    if (vec && part) {
+        for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
+            const float* src = part + (size_t)r * ldz + c;
+            float4 v = *reinterpret_cast<const float4*>(src);
+            for (int s0 = 1; s0 < n_splits; s0 += 8) {             // eight splits' loads in flight; the adds stay in split order
+                float4 t[8];
+#pragma unroll
+                for (int k = 0; k < 8; ++k) t[k] = *reinterpret_cast<const float4*>(src + (size_t)min(s0 + k, n_splits - 1) * split_stride);
+#pragma unroll
+                for (int k = 0; k < 8; ++k)
+                    if (s0 + k < n_splits) { v.x += t[k].x; v.y += t[k].y; v.z += t[k].z; v.w += t[k].w; }
+            }
+            *reinterpret_cast<float4*>(pn_row + c) = v;
+            count(v.x); count(v.y); count(v.z); count(v.w);
+        }
+    } else if (vec) {
+        for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+            union { uint4 raw; T e[VEC]; } v;
+            v.raw = *reinterpret_cast<const uint4*>(z_rows + (size_t)r * ldz + c);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) {
+                const float f = to_f32(v.e[k]);
+                pn_row[c + k] = f;
+                count(f);
+            }
+        }
+    } else {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) {
+            float v;
+            if (part) {
+                v = part[(size_t)r * ldz + c];
+                for (int s = 1; s < n_splits; ++s) v += part[(size_t)s * split_stride + (size_t)r * ldz + c];
+            } else {
+                v = to_f32(z_rows[(size_t)r * ldz + c]);
+            }
+            pn_row[c] = v;
+            count(v);
+        }
+    }
+    const float n = (float)width;
+    const float f1 = coef[0] / sqrtf(block_sum(s2, red0) / n + eps);
+    const float f2 = coef[1] / sqrtf(block_sum(s4, red1) / n + eps);
+    const float f3 = coef[2] / sqrtf(block_sum(s6, red2) / n + eps);
+    const float e = coef[3];
+    auto act = [&](float v) { return fmaf(v, fmaf(v, fmaf(v, f3, f2), f1), e); };
+    T* o = out + (size_t)r * ldo;
+    if (vec) {
+        for (int c = threadIdx.x * VEC; c < width; c += blockDim.x * VEC) {
+            union { uint4 raw; T e[VEC]; } v;
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) v.e[k] = from_f32<T>(act(pn_row[c + k]));
+            *reinterpret_cast<uint4*>(o + c) = v.raw;
+        }
+    } else {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) o[c] = from_f32<T>(act(pn_row[c]));
+    }
+}
+
+extern "C" int cml_poly_norm(const float* part, int n_splits, long split_stride, long ldz, const void* z_rows, int dtype,
+                             const float* coef, float eps, void* out, long ldo, int rows, int width, void* stream) {
+    if (rows <= 0) return 0;
+    if (width < 1 || (part ? n_splits < 1 : z_rows == nullptr)) return CML_ERR_BAD_SIZE;
+    const size_t smem = (size_t)((width + 3) & ~3) * sizeof(float);
+    if (smem > 200 * 1024) return CML_ERR_BAD_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int block = width >= 4096 ? 512 : (width >= 1024 ? 256 : 128);
+#define PLN_CASE(T_, D_)                                                                                                  \
+    if (dtype == D_) {                                                                                                    \
+        if (smem > 48 * 1024 && cml_allow_smem<poly_norm_kernel<T_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE;       \
+        launch_pdl(poly_norm_kernel<T_>, dim3(rows), dim3(block), smem, s, part, n_splits, split_stride, ldz,            \
+                   (const T_*)z_rows, coef, eps, (T_*)out, ldo, width);                                                   \
+        return cml_launch_status();                                                                                       \
+    }
+    PLN_CASE(float, CML_DTYPE_F32)
+    PLN_CASE(bf16, CML_DTYPE_BF16)
+#undef PLN_CASE
+    return CML_ERR_BAD_DTYPE;
+}
+
+// out[r, c] = tanh(sum over splits of z[split][r, col0 + c]) in the compute type: the narrow middle of a low-rank pair.
+template <typename T>
+__global__ void tanh_columns_kernel(const float* __restrict__ z, long ldz, int n_splits, long split_stride, int col0,
+                                    T* __restrict__ out, long n, int width) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const long r = i / width;
+    const float* src = z + r * ldz + col0 + (i - r * width);
+    float v = src[0];
+    for (int s = 1; s < n_splits; ++s) v += src[(size_t)s * split_stride];
+    out[i] = from_f32<T>(tanhf(v));
+}
+
+extern "C" int cml_tanh_columns(const float* z, long ldz, int n_splits, long split_stride, int col0, void* out, int dtype, int rows,
+                                int width, void* stream) {
+    const long n = (long)rows * width;
+    if (n <= 0) return 0;
+    if (n_splits < 1 || col0 < 0) return CML_ERR_BAD_SIZE;
+    const dim3 grid((unsigned)((n + 255) / 256));
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == CML_DTYPE_F32) launch_pdl(tanh_columns_kernel<float>, grid, dim3(256), 0, s, z, ldz, n_splits, split_stride, col0, (float*)out, n, width);
+    else if (dtype == CML_DTYPE_BF16) launch_pdl(tanh_columns_kernel<bf16>, grid, dim3(256), 0, s, z, ldz, n_splits, split_stride, col0, (bf16*)out, n, width);
+    else return CML_ERR_BAD_DTYPE;
+    return cml_launch_status();
+}
+
 // x[r, c] *= sigmoid(gate[r, gate_col + c]) in place (x in the compute type, gate float).
 template <typename T>
 __global__ void gate_rows_kernel(T* __restrict__ x, const float* __restrict__ gate, long ldg, int gate_col, long n, int width) {

@@ -3,6 +3,8 @@
 residual stream stays float32; mixer and feed-forward add into it in place."""
 from __future__ import annotations
 
+import torch
+
 from .base import Part, build_part, register_part
 
 
@@ -205,3 +207,89 @@ class PostNormBlock(Part):
             x = self.norm2.sum_normed(ctx, y, h, self.alpha, bias)
         if self.after is not None:
             self.after.forward(ctx, x, h)
+
+
+@register_part("block", "parallel")
+class ParallelBlock(Part):
+    """Both sublayers read the same stream, each through a norm of its own: x += mixer(norm1(x)) + ffn(norm2(x)). The two
+    norms run in one pass over the rows where they can. Where mixer and feed-forward both end in one matrix and can hand
+    over the rows that go into it (``output_weight()`` and ``output_rows(ctx, x, out)``), those rows stand side by side and
+    one product with the two matrices side by side makes and adds both outputs; otherwise each adds into the stream
+    itself. A layer without a feed-forward has only the first sublayer."""
+
+    def __init__(self, layer_spec):
+        super().__init__({}, "")
+        from ..errors import ConfigError
+        self.norm1 = build_part("norm", layer_spec.norm1)
+        self.mixer = build_part("mixer", layer_spec.mixer)
+        self.ffn = build_part("ffn", layer_spec.ffn) if layer_spec.ffn is not None else None
+        if self.ffn is not None and layer_spec.norm2 is None:
+            raise ConfigError("block.arrangement", "the parallel arrangement needs norm2 with a feed-forward")
+        self.norm2 = build_part("norm", layer_spec.norm2) if self.ffn is not None else None
+        self.w_joint = None
+
+    def parts(self):
+        return tuple(p for p in (self.norm1, self.mixer, self.norm2, self.ffn) if p is not None)
+
+    def tensor_specs(self):
+        out = {}
+        for p in self.parts():
+            out.update(p.tensor_specs())
+        return out
+
+    def load(self, tensors, device, dtype):
+        for p in self.parts():
+            p.load(tensors, device, dtype)
+        self.w_joint = None
+        if self.ffn is not None and hasattr(self.mixer, "output_weight") and hasattr(self.ffn, "output_weight"):
+            a, b = self.mixer.output_weight(), self.ffn.output_weight()
+            if a is not None and b is not None:
+                # the matrices' columns side by side; each part keeps its own as a view
+                self.w_joint = torch.cat([a, b], dim=1).contiguous()
+                self.mixer.set_output_weight(self.w_joint[:, :a.shape[1]])
+                self.ffn.set_output_weight(self.w_joint[:, a.shape[1]:])
+
+    @property
+    def graph_safe(self):
+        return all(p.graph_safe for p in self.parts())
+
+    @property
+    def graph_safe_any_step(self):
+        return all(p.graph_safe_any_step for p in self.parts())
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def query_tile_sizes(self):
+        return self.mixer.query_tile_sizes()
+
+    def _normed(self, ctx, h):
+        """The rows of both norms (the second None without a feed-forward)."""
+        if not self.norm1.handles_pending:
+            ctx.settle(h)
+        if self.ffn is None:
+            return self.norm1.forward(ctx, h), None
+        pair = self.norm1.pair_normed(ctx, h, self.norm2) if hasattr(self.norm1, "pair_normed") else None
+        if pair is not None:
+            return pair
+        ctx.settle(h)
+        # the second norm's rows wait under a name of their own while the mixer works
+        return self.norm1.forward(ctx, h), self.norm2.forward(ctx, h, name="normed_b")
+
+    def forward(self, ctx, h):
+        ctx.rows_copy = None
+        x, x2 = self._normed(ctx, h)
+        if self.w_joint is not None:
+            n_a = self.mixer.output_weight().shape[1]
+            rows = ctx.buffer("joint_rows", (ctx.n_rows, self.w_joint.shape[1]))
+            self.mixer.output_rows(ctx, x, rows[:, :n_a])
+            self.ffn.output_rows(ctx, x2, rows[:, n_a:])
+            from . import linear
+            linear.add_into_residual(ctx, rows, self.w_joint, h, "joint_partial")
+            return
+        for part, rows in ((self.mixer, x), (self.ffn, x2)):
+            if part is None:
+                continue
+            if not part.handles_pending:
+                ctx.settle(h)
+            part.forward(ctx, rows, h)

@@ -15,7 +15,9 @@ identity] is added to the scores for the choice alone (the weights use the score
 the experts (identity ones included) form ``count`` equal groups of neighbours, a group's score is its largest choice
 score, and only experts of the ``keep`` best groups can be chosen; ``route_scale`` multiplies the weights; ``gate_act``
 and ``shared_gate_act`` (alpha, limit, shift): the experts' gated activation min(g, limit) sigmoid(alpha min(g, limit))
-(clamp(u, +-limit) + shift) instead of silu(g) u.
+(clamp(u, +-limit) + shift) instead of silu(g) u; ``router_bias``: a tensor ``router.b`` [experts + identity] is part of the
+logits; ``shared_output_gate``: the shared expert's output times sigmoid(x . ``shared.sg``), one number per row. A softmax
+over all experts that is renormalized over the chosen ones is the softmax over the chosen logits.
 
 Tensors under the prefix: ``router`` [experts, hidden]; per expert ``e<i>.gate``, ``e<i>.up`` [ff, hidden] and
 ``e<i>.down`` [hidden, ff]; the shared expert's under ``shared.`` with the same three names. The experts'
@@ -49,6 +51,7 @@ class RoutedExperts(Part):
         self.routed = self.experts + self.identity          # outputs of the router
         self.correction = bool(params.get("correction", False))
         self.groups, self.keep_groups = (int(v) for v in (params.get("groups") or (1, 1)))
+        self.router_bias = bool(params.get("router_bias", False))
         self.route_scale = float(params["route_scale"]) if params.get("route_scale") is not None else 1.0
         self.act = ops.GateAct(*params["gate_act"]) if params.get("gate_act") else None
         self.top = int(params["top"])
@@ -77,13 +80,18 @@ class RoutedExperts(Part):
                                                                 "intermediate_size": int(params["shared_size"]),
                                                                 "names": ("gate", "up", "down"),
                                                                 "gate_act": params.get("shared_gate_act")}, prefix + "shared."))
-        self.w_router = self.w_gate = self.w_up = self.w_down = self.w_correction = None
+        self.shared_gate = bool(params.get("shared_output_gate", False)) and self.shared is not None
+        self.w_router = self.w_gate = self.w_up = self.w_down = self.w_correction = self.b_router = None
 
     def tensor_specs(self):
         p, hid = self.prefix, self.hidden_size
         specs = {p + "router": TensorSpec((self.routed, hid))}
         if self.correction:
             specs[p + "correction"] = TensorSpec((self.routed,), "choice_bias")
+        if self.router_bias:
+            specs[p + "router.b"] = TensorSpec((self.routed,), "input_bias")
+        if self.shared_gate:
+            specs[p + "shared.sg"] = TensorSpec((1, hid))
         for e in range(self.experts):
             specs[f"{p}e{e}.gate"] = TensorSpec((self.ff, hid))
             specs[f"{p}e{e}.up"] = TensorSpec((self.ff, hid))
@@ -95,6 +103,10 @@ class RoutedExperts(Part):
     def load(self, tensors, device, dtype):
         p = self.prefix
         self.w_router = to_device(tensors[p + "router"], device, dtype)
+        if self.router_bias:
+            self.b_router = tensors[p + "router.b"].to(device=device, dtype=torch.float32).contiguous()
+        if self.shared_gate:            # one more row of the router's product
+            self.w_router = torch.cat([self.w_router, to_device(tensors[p + "shared.sg"], device, dtype)], 0).contiguous()
         if self.correction:
             self.w_correction = tensors[p + "correction"].to(device=device, dtype=torch.float32).contiguous()
         stack = lambda n: torch.stack([to_device(tensors[f"{p}e{e}.{n}"], device, dtype)       # noqa: E731
@@ -108,16 +120,20 @@ class RoutedExperts(Part):
         if self.shared is not None:
             self.shared.load(tensors, device, dtype)
 
-    def output(self, ctx, x, name: str, stream=None):
+    def output(self, ctx, x, name: str, stream=None, into=None):
         """(y, None): float32 [rows, hidden] in the step's buffer ``name``. ``stream``: the rows of ``x`` in float32
-        where the caller has them (what an identity expert hands back); else ``x`` itself."""
+        where the caller has them (what an identity expert hands back); else ``x`` itself. ``into`` (float32 [rows,
+        hidden]): the output is added to these rows instead."""
         rows, top, E = x.shape[0], self.top, self.routed
         pairs = rows * top
         i32 = lambda n, k: ctx.buffer(f"{name}_{n}", (k,), torch.int32)        # noqa: E731
         logits = linear.product_f32(ctx, x, self.w_router, name + "_router")          # split sums where the step has few rows
+        shared_gate = None
+        if self.shared_gate:
+            logits, shared_gate = logits[..., :E], logits[..., E:]
         ids, wts = i32("ids", pairs), ctx.buffer(name + "_wts", (pairs,), torch.float32)
         ops.route_topk(logits, top, self.scoring == "softmax", self.renormalize, ids, wts, self.w_correction, self.groups,
-                       self.keep_groups, self.route_scale)
+                       self.keep_groups, self.route_scale, self.b_router)
         rank, counts, offsets, tile_first = i32("rank", pairs), i32("counts", E), i32("offsets", E + 1), i32("tiles", E + 1)
         tc = self.w_gate_up is not None
         ops.expert_plan(ids, E, rank, counts, offsets, tile_first, ops.EXPERT_TILE_ROWS_TC if tc else ops.EXPERT_TILE_ROWS)
@@ -133,12 +149,12 @@ class RoutedExperts(Part):
             ops.expert_gemm(xs, self.w_gate, self.w_up, act, offsets, tile_first, self.act)
             ops.expert_gemm(act, self.w_down, None, ys, offsets, tile_first)
         shared = self.shared.output(ctx, x, name + "_shared")[0] if self.shared is not None else None
-        out = ctx.buffer(name, (rows, self.hidden_size), torch.float32)
+        out = into if into is not None else ctx.buffer(name, (rows, self.hidden_size), torch.float32)
         same = (ids, self.experts, stream if stream is not None else x) if self.identity else None
-        ops.expert_combine(ys, place, wts, top, self.weight_on == "output", shared, out, same)
+        ops.expert_combine(ys, place, wts, top, self.weight_on == "output", shared, out, same, shared_gate,
+                           into is not None)
         return out, None
 
     def forward(self, ctx, x, residual):
-        y, _ = self.output(ctx, x, "experts_out")
-        ctx.settle(residual)
-        ops.add_partials(residual, y.unsqueeze(0))
+        # (whatever is still pending or deferred for the stream is added by its next reader, before or after this)
+        self.output(ctx, x, "experts_out", into=residual)

@@ -61,7 +61,9 @@ class SwiGLU(Part):
 @register_part("ffn", "dense")
 class DenseFeedForward(Part):
     """d = act(x Wu^T + bu) Wd^T + bd. ``activation``: "gelu_tanh" (the tanh form of GELU), "gelu_erf" (the exact one,
-    0.5 z (1 + erf(z / sqrt 2))) or "relu_squared" (max(z, 0)^2); ``bias``: whether the two projections have biases (``up.b``, ``down.b``). Tensors ``up``
+    0.5 z (1 + erf(z / sqrt 2))), "relu_squared" (max(z, 0)^2) or "poly_norm" (a N(z) + b N(z^2) + c N(z^3) + e with the four
+    numbers of the tensor ``act``; powers element by element, N divides a row by its root mean square with ``eps``; no
+    biases); ``bias``: whether the two projections have biases (``up.b``, ``down.b``). Tensors ``up``
     [intermediate, hidden] and ``down`` [hidden, intermediate] under the prefix."""
     graph_safe = True
     graph_safe_any_step = True
@@ -73,11 +75,18 @@ class DenseFeedForward(Part):
         self.hidden_size = int(params["hidden_size"])
         self.intermediate_size = int(params["intermediate_size"])
         self.activation = params.get("activation") or self.default_activation
-        if self.activation not in ("gelu_tanh", "gelu_erf", "relu_squared"):
-            from ..errors import ConfigError
-            raise ConfigError("activation", f"unknown activation {self.activation!r}; known: gelu_tanh, gelu_erf, relu_squared")
-        self.act = ops.ACTIVATIONS[self.activation]
+        from ..errors import ConfigError
+        if self.activation not in ("gelu_tanh", "gelu_erf", "relu_squared", "poly_norm"):
+            raise ConfigError("activation", f"unknown activation {self.activation!r}; known: gelu_tanh, gelu_erf, relu_squared, poly_norm")
+        self.poly = self.activation == "poly_norm"
+        self.act = None if self.poly else ops.ACTIVATIONS[self.activation]
         self.bias = bool(params.get("bias", False))
+        self.eps = float(params.get("eps", 1e-6))
+        if self.poly and self.bias:
+            raise ConfigError("bias", "the activation poly_norm goes with projections without biases")
+        if self.poly and self.intermediate_size > 51200:
+            raise ConfigError("intermediate_size", f"the poly_norm kernel takes rows of up to 51,200 values, got {self.intermediate_size}")
+        self.coef = None
         self.w_up = self.w_down = self.b_up = self.b_down = None
 
     def tensor_specs(self):
@@ -87,20 +96,41 @@ class DenseFeedForward(Part):
         if self.bias:
             specs[p + "up.b"] = TensorSpec((self.intermediate_size,), "input_bias")
             specs[p + "down.b"] = TensorSpec((self.hidden_size,), "input_bias")
+        if self.poly:
+            specs[p + "act"] = TensorSpec((4,), "fraction")
         return specs
 
     def load(self, tensors, device, dtype):
         import torch
+        if self.poly:
+            self.coef = tensors[self.prefix + "act"].to(device=device, dtype=torch.float32).contiguous()
         self.w_up = to_device(tensors[self.prefix + "up"], device, dtype)
         self.w_down = to_device(tensors[self.prefix + "down"], device, dtype)
         if self.bias:
             self.b_up = tensors[self.prefix + "up.b"].to(device=device, dtype=torch.float32).contiguous()
             self.b_down = tensors[self.prefix + "down.b"].to(device=device, dtype=torch.float32).contiguous()
 
-    def _activations(self, ctx, x, name="ffn_act"):
-        act = ctx.buffer(name, (x.shape[0], self.intermediate_size))
+    def _activations(self, ctx, x, name="ffn_act", out=None):
+        act = out if out is not None else ctx.buffer(name, (x.shape[0], self.intermediate_size))
+        if self.poly:
+            part = linear.partial_sums(ctx, x, self.w_up, "up_partial")
+            if part is None:
+                linear.linear(ctx, x, self.w_up, act, linear.STORE)
+            ops.poly_norm(act if part is None else part, self.coef, self.eps, act)
+            return act
         linear.product_act(ctx, x, self.w_up, act, "up_partial", act=self.act, bias=self.b_up)
         return act
+
+    # a block may put the rows that go into ``down`` beside a mixer's and run one product for both (``act``'s other
+    # forms write whole contiguous rows)
+    def output_weight(self):
+        return self.w_down if self.poly else None
+
+    def set_output_weight(self, w):
+        self.w_down = w
+
+    def output_rows(self, ctx, x, out):
+        self._activations(ctx, x, out=out)
 
     def forward(self, ctx, x, residual):
         act = self._activations(ctx, x)

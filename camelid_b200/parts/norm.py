@@ -1,6 +1,7 @@
 """RMSNorm: y = x * rsqrt(mean(x^2) + eps) * w in float32 (src/tensor/mod.rs:2086-2096;
 device twins rms_norm_f32 and rms_norm_batched at src/cuda_resident.rs:89, :1925). The
-input is the float32 residual stream; the output has the compute type."""
+input is the float32 residual stream; the output has the compute type. ``offset`` (default 0) is added to the
+stored weight: 1 for weights stored around zero (the sum is kept in float32)."""
 from __future__ import annotations
 
 import torch
@@ -21,13 +22,17 @@ class RMSNorm(Part):
         self.hidden_size = int(params["hidden_size"])
         self.eps = float(params["eps"])
         self.tensor = params.get("tensor") or self.prefix + "weight"      # the weight's full name
+        self.offset = float(params.get("offset") or 0.0)
         self.weight = None
 
     def tensor_specs(self):
-        return {self.tensor: TensorSpec((self.hidden_size,), "norm")}
+        return {self.tensor: TensorSpec((self.hidden_size,), "centred_norm" if self.offset == 1.0 else "norm")}
 
     def load(self, tensors, device, dtype):
         w = tensors[self.tensor]
+        if self.offset:
+            self.weight = to_device(w, device, torch.float32) + self.offset
+            return
         # a weight stored in 32-bit stays so; a 16-bit one becomes float32 only on the float32 path
         keep = None if w.dtype == torch.float32 else dtype
         self.weight = to_device(w, device, keep)
@@ -46,6 +51,19 @@ class RMSNorm(Part):
         pending, ctx.pending = ctx.pending, None            # split sums still to be added to h: added here
         ops.rmsnorm(h, self.weight, self.eps, out, rows_index, pending)
         return out
+
+    def pair_normed(self, ctx, h, other, name="normed", other_name="normed_b"):
+        """(rows of this norm, rows of ``other``) of the same stream rows, in one pass where the two norms differ in their
+        weights alone (else None: the caller runs both)."""
+        if not (type(other) is type(self) and other.weight.dtype == self.weight.dtype and other.hidden_size == self.hidden_size
+                and other.eps == self.eps):
+            return None
+        a, b = ctx.buffer(name, h.shape), ctx.buffer(other_name, h.shape)
+        if ctx.deferred is not None:
+            linear.run_deferred(ctx)
+        pending, ctx.pending = ctx.pending, None
+        ops.rmsnorm(h, self.weight, self.eps, a, None, pending, other.weight, b)
+        return a, b
 
     def sum_normed(self, ctx, y, residual, alpha: float = 1.0, bias=None):
         """residual = rmsnorm(alpha * residual + y + bias) * w in place: this norm *after* a residual sum, where the

@@ -32,6 +32,8 @@ pairs a1/a2, g1/g2 or the plain matrices a, g) and ``gate`` "sigmoid" | "silu".
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..cache.book import StateSpec
@@ -300,3 +302,101 @@ class Retention(Part):
 
     def branch_output(self, ctx, x, name: str, proj=None):
         return linear.product_f32(ctx, self.read_out(ctx, x), self.w_o, name)
+
+
+@register_part("mixer", "general_delta")
+class GeneralDelta(Part):
+    """The delta rule with a decay w and a removal rate a per key channel. r, k (``num_heads`` x ``key_dim``) and v
+    (``num_heads`` x ``value_dim``) are plain projections, u = k / sqrt(sum k^2 + 1e-6) per head,
+
+        w = exp(-rate * sigmoid(W2 tanh(W1 x) + w0)),   a = sigmoid(Wa x + ba),
+        S_t = diag(w) S_(t-1) - (a * u) (u^T S_(t-1)) + k v^T,   o_t = S_t^T r
+
+    both terms of the write on the old state. o is divided by its root mean square per head; the heads side by side are
+    multiplied by ``norm`` (all heads' size) and sigmoid(Wg x) and projected by Wo. S is float32 per sequence and head, zero at
+    the start; decays, rates, unit keys, the scan and the norm are float32. ``decay_rate``: the factor of the decay's exponent
+    (default exp(-1/2)). The width of the decays' narrow input is the stored tensors' own. Tensors ``r k v a a.b g w1 w2 w0
+    norm o``."""
+    graph_safe = True
+    graph_safe_any_step = True
+    FEW_ROWS = 32                   # up to here a step makes W2 tanh(.) in the kernel that prepares the scan's rows
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.hidden_size = int(params["hidden_size"])
+        self.eps = float(params.get("eps", 1e-6))
+        self.num_heads = int(params["num_heads"])
+        self.key_dim = int(params["key_dim"])
+        self.value_dim = int(params.get("value_dim") or self.key_dim)
+        self.decay_rate = float(params["decay_rate"]) if params.get("decay_rate") is not None else math.exp(-0.5)
+        _check_dims(self.key_dim, self.value_dim)
+        self.rank = int(params.get("rank") or max(8, self.hidden_size // 16 // 8 * 8))      # for random weights
+        self.k_width = self.num_heads * self.key_dim
+        self.v_width = self.num_heads * self.value_dim
+        self.gate_col = 3 * self.k_width + self.v_width               # columns of the input product: r, k, v, a, g, w1
+        self.narrow_col = self.gate_col + self.v_width
+        self.w_in = self.w2 = self.w_o = self.a_bias = self.w0 = self.norm_w = None
+
+    def tensor_specs(self):
+        p, hid, K, V = self.prefix, self.hidden_size, self.k_width, self.v_width
+        return {p + "r": TensorSpec((K, hid)), p + "k": TensorSpec((K, hid)), p + "v": TensorSpec((V, hid)),
+                p + "a": TensorSpec((K, hid)), p + "a.b": TensorSpec((K,), "input_bias"), p + "g": TensorSpec((V, hid)),
+                p + "w1": TensorSpec((self.rank, hid), "linear", (0,)), p + "w2": TensorSpec((K, self.rank), "low_rank", (1,)),
+                p + "w0": TensorSpec((K,), "log_rate"), p + "norm": TensorSpec((V,), "norm"), p + "o": TensorSpec((hid, V))}
+
+    def load(self, tensors, device, dtype):
+        p = self.prefix
+        dev = lambda n: to_device(tensors[p + n], device, dtype)                                  # noqa: E731
+        f32 = lambda n: tensors[p + n].to(device=device, dtype=torch.float32).contiguous()      # noqa: E731
+        w1, w2 = dev("w1"), dev("w2")
+        if w2.shape[1] != w1.shape[0]:
+            raise WeightsError(wrong_shape=[(p + "w2", (self.k_width, w1.shape[0]), tuple(w2.shape))])
+        pad = -w1.shape[0] % 8                      # zeros: what the tensor-core product takes is a multiple of 8
+        if pad:
+            w1 = torch.cat([w1, w1.new_zeros((pad, w1.shape[1]))], 0)
+            w2 = torch.cat([w2, w2.new_zeros((w2.shape[0], pad))], 1)
+        self.w_in = torch.cat([dev(n) for n in ("r", "k", "v", "a", "g")] + [w1], 0).contiguous()
+        self.w2, self.w_o = w2.contiguous(), dev("o")
+        self.a_bias, self.w0, self.norm_w = f32("a.b"), f32("w0"), f32("norm")
+
+    def cache_spec(self):
+        return StateSpec((self.num_heads, self.value_dim, self.key_dim), "float32", "delta")
+
+    def read_out(self, ctx, x, out=None):
+        n, H, D, V = ctx.n_rows, self.num_heads, self.key_dim, self.value_dim
+        sums = linear.product_f32(ctx, x, self.w_in, "gd_proj")            # split sums where the step is small: added below
+        packed = ctx.buffer("gd_packed", (n, H, 4 * D + V), torch.float32)
+        scal = ctx.buffer("gd_scalars", (n, H, 4), torch.float32)
+        split = sums.dim() == 3
+        gate, gate_col, high = sums, self.gate_col, None
+        if split:
+            gate, gate_col = ctx.buffer("gd_gate", (n, self.v_width), torch.float32), 0
+        if n > self.FEW_ROWS:
+            low = ctx.buffer("gd_low", (n, self.w2.shape[1]))
+            ops.tanh_columns(sums, self.narrow_col, low)
+            high = linear.product_f32(ctx, low, self.w2, "gd_high")
+        ops.delta_inputs(sums, self.a_bias, self.w0, self.decay_rate, packed, scal, H, D, V, high, None if high is not None else self.w2,
+                         gate if split else None)
+        raw = ctx.buffer("gd_raw", (n, self.v_width), torch.float32)
+        ops.general_delta_scan(packed, scal, ctx.state("delta"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, raw,
+                               ctx.n_seqs, H, D, V)
+        if out is None:
+            out = ctx.buffer("gd_out", (n, self.v_width))
+        ops.head_norm_gate(raw, False, self.norm_w, True, gate, gate_col, out, H, V, self.eps)
+        return out
+
+    def forward(self, ctx, x, residual):
+        linear.add_into_residual(ctx, self.read_out(ctx, x), self.w_o, residual, "o_partial")
+
+    def branch_output(self, ctx, x, name: str, proj=None):
+        return linear.product_f32(ctx, self.read_out(ctx, x), self.w_o, name)
+
+    # a block may put the rows that go into ``o`` beside a feed-forward's and run one product for both
+    def output_weight(self):
+        return self.w_o
+
+    def set_output_weight(self, w):
+        self.w_o = w
+
+    def output_rows(self, ctx, x, out):
+        self.read_out(ctx, x, out)

@@ -24,10 +24,11 @@ STD = 0.02
 # init rule -> (mean, standard deviation). Besides matrices and norm weights: small positive
 # numbers (mixing weights, rates of a distance penalty), gate biases that keep a memory
 # (forget) or leave it alone (input), logarithms of decay rates and their step-size biases,
-# taps of a short convolution.
+# taps of a short convolution, norm weights stored around zero.
 INIT = {"linear": (0.0, STD), "embedding": (0.0, STD), "norm": (1.0, STD), "fraction": (0.3, 0.05),
         "forget_bias": (4.0, 0.5), "input_bias": (0.0, 0.3), "log_rate": (-2.0, 0.5), "conv": (0.25, 0.3),
-        "low_rank": (0.0, 0.1), "choice_bias": (0.0, 0.02)}
+        "low_rank": (0.0, 0.1), "choice_bias": (0.0, 0.02),
+        "centred_norm": (0.0, STD)}
 
 
 def mean_of(init: str) -> float:
