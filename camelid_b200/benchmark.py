@@ -908,6 +908,146 @@ def run_kizezen(sizes=("small", "medium"), batch: int = 8, prompt_tokens: int = 
     return out
 
 
+RAMOPEL_SIZES = {
+    # width, layers (attention over a latent with a dense feed-forward and generalized delta rule with a routed one, in
+    # turn; every second attention reads the latent rows of the one before it), feed-forward size, heads of `head` channels
+    # in both mixers, the turned part, the two latents, the window, experts / choices / expert size / shared expert size
+    "small": dict(width=1024, layers=8, ff=4096, heads=8, head=128, rot=64, rank=512, q_rank=512, window=512, experts=16, top=2,
+                  expert_ff=1024, shared_ff=1024, narrow=64, vocab=32768),
+    "medium": dict(width=2048, layers=16, ff=8192, heads=16, head=128, rot=64, rank=512, q_rank=768, window=1024, experts=32, top=4,
+                   expert_ff=1024, shared_ff=1024, narrow=96, vocab=32768),
+    "wide": dict(width=4096, layers=8, ff=14336, heads=32, head=128, rot=64, rank=512, q_rank=1536, window=1024, experts=32, top=4,
+                 expert_ff=2048, shared_ff=2048, narrow=128, vocab=32768),
+}
+
+
+def ramopel_config_for(size: str) -> dict:
+    s = RAMOPEL_SIZES[size]
+    H, D, R = s["heads"], s["head"], s["rot"]
+    latent = {"heads": H, "dim": D, "rot_dim": R, "vdim": D, "kv_rank": s["rank"], "q_rank": s["q_rank"], "scale": (D + R) ** -0.5,
+              "mask": {"size": s["window"]}, "rot": {"base": 10000.0, "dims": R}}
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "top": s["top"]}, "expert": {"ff": s["expert_ff"], "limit": 7.0},
+           "shared": {"ff": s["shared_ff"], "limit": 7.0}}
+    layers = []
+    for i in range(s["layers"]):
+        if i % 2 == 0:
+            more = {"kv_from": i - 2} if i % 4 == 2 else {}
+            layers.append({"type": "latent_attention", "mixer": {**latent, **more}, "mlp": {"kind": "dense", "ff": s["ff"]}})
+        else:
+            layers.append({"type": "general_delta", "mixer": {"heads": H, "dim": D, "rank": s["narrow"]}, "mlp": copy.deepcopy(moe)})
+    return {"architecture": "Ramopel", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "layers": layers}
+
+
+def kizezen_config_like_ramopel(size: str) -> dict:
+    """The Kizezen decoder of the same width, depth, heads, latent and vocabulary, attention over a latent and retention
+    in turn (the library's closest model: the same attention, a matrix state per head), every feed-forward dense; where
+    the other has routed experts, the feed-forward whose matrices have as many elements as a token passes there."""
+    s = RAMOPEL_SIZES[size]
+    H, D = s["heads"], s["head"]
+    latent = {"dim": D, "rot_dim": s["rot"], "vdim": D, "heads": H, "kv_rank": s["rank"], "scale": (D + s["rot"]) ** -0.5,
+              "rot": {"dims": s["rot"], "base": 10000.0}}
+    retention = {"dim": D, "vdim": D, "heads": H, "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * i / max(H - 1, 1)) for i in range(H)]}
+    routed_ff = 3 * (s["top"] * s["expert_ff"] + s["shared_ff"]) // 2
+    layers = [{"type": "latent_attention", "mixer": dict(latent), "mlp": {"kind": "dense", "ff": s["ff"]}} if i % 2 == 0 else
+              {"type": "retention", "mixer": dict(retention), "mlp": {"kind": "dense", "ff": routed_ff}} for i in range(s["layers"])]
+    return {"architecture": "Kizezen", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "layers": layers}
+
+
+def _ramopel_matrices(L: dict, W: int, experts: float) -> float:
+    """Elements of the matrices a step passes in one layer, with ``experts`` routed ones."""
+    m, f = L["mixer"], L.get("mlp")
+    H, D = m["heads"], m["dim"]
+    if L["type"] == "latent_attention":
+        n = W * m["q_rank"] + m["q_rank"] * H * (D + m["rot_dim"]) + H * (D + m["vdim"]) * m["kv_rank"] + H * m["vdim"] * W
+        if m.get("kv_from") is None:
+            n += W * (m["kv_rank"] + m["rot_dim"])
+    else:
+        n = 6 * W * H * D + m["rank"] * (W + H * D)
+    if f and f["kind"] == "dense":
+        n += 2 * W * f["ff"]
+    elif f:
+        n += W * f["router"]["experts"] + 3 * W * experts * f["expert"]["ff"]
+        if f.get("shared"):
+            n += 3 * W * f["shared"]["ff"] + W
+    return n
+
+
+def ramopel_step_bytes(cfg: dict, batch: int, context: float, elem: int) -> dict:
+    """Bytes a decode step must move: every matrix once (of the routed experts as many as ``batch`` rows reach on average
+    when their choices are uniform; the output head, no embedding table), per attention one latent row for every visible
+    position, every delta state read and written in float32."""
+    W = cfg["width"]
+    weights = kv = state = 0.0
+    for L in cfg["layers"]:
+        m, f = L["mixer"], L.get("mlp")
+        reached = 0.0
+        if f and f["kind"] == "moe":
+            r = f["router"]
+            reached = r["experts"] * (1.0 - (1.0 - r["top"] / r["experts"]) ** batch)
+        weights += _ramopel_matrices(L, W, reached)
+        if L["type"] == "latent_attention":
+            seen = min(context, m["mask"]["size"]) if m.get("mask") else context
+            kv += batch * seen * (m["kv_rank"] + m["rot_dim"])
+        else:
+            state += 2.0 * batch * m["heads"] * m["dim"] * m["dim"] * 4
+    weights += cfg["vocab"] * W
+    return {"weights": int(weights * elem), "kv": int(kv * elem), "state": int(state), "total": int((weights + kv) * elem + state)}
+
+
+def ramopel_prefill_flops(cfg: dict, tokens: int) -> float:
+    """2 x tokens x (elements of every matrix a token passes, ``top`` routed experts and the latent's maps among them)
+    plus the attention over the visible keys (per head and pair of positions the key's and the value's channels) and 6
+    flops per element of a delta state and token (the removal's product, the write, the read-out)."""
+    W = cfg["width"]
+    total = 0.0
+    for L in cfg["layers"]:
+        m, f = L["mixer"], L.get("mlp")
+        total += 2.0 * tokens * _ramopel_matrices(L, W, f["router"]["top"] if f and f["kind"] == "moe" else 0)
+        if L["type"] == "latent_attention":
+            window = m["mask"]["size"] if m.get("mask") else tokens
+            total += 2.0 * sum(min(i + 1, window) for i in range(tokens)) * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"])
+        else:
+            total += 6.0 * tokens * m["heads"] * m["dim"] * m["dim"]
+    return total + 2.0 * W * cfg["vocab"]
+
+
+def run_ramopel(sizes=("small", "medium"), batch: int = 8, prompt_tokens: int = 512, steps: int = 64, warmup: int = 4,
+                prefill_tokens: int = 2048, dtype: str = "bfloat16") -> dict:
+    """Decode steps (timed on the device in the loop ``generate`` runs) and prefill steps of the Ramopel decoder and of
+    the Kizezen decoder of equal width, depth, heads, latent and vocabulary, random weights."""
+    from . import api
+    pk = peaks()
+    elem = 2 if dtype == "bfloat16" else 4
+    out = {"metric": "decode and prefill tokens/s, Ramopel beside the Kizezen decoder of equal size", "dtype": dtype,
+           "batch": batch, "prompt_tokens": prompt_tokens, "steps": steps, "warmup": warmup,
+           "prefill_tokens": prefill_tokens, "peaks": pk["source"], "data": "synthetic (seeded uniform token ids, random weights)",
+           "sizes": {}}
+    for size in sizes:
+        rec = {"shape": RAMOPEL_SIZES[size]}
+        for label, cfg in (("ramopel", ramopel_config_for(size)), ("kizezen", kizezen_config_like_ramopel(size))):
+            lm = api.from_random(cfg, seed=7, dtype=dtype)
+            vocab = {"vocab_size": RAMOPEL_SIZES[size]["vocab"]}
+            rng = np.random.default_rng(7)
+            dec = measure_decode_device(lm, vocab, batch, prompt_tokens, steps, warmup, rng)
+            bytes_step = (ramopel_step_bytes if label == "ramopel" else kizezen_step_bytes)(cfg, batch, dec["context"], elem)
+            pre = measure_prefill(lm, vocab, prefill_tokens, rng)
+            flops = (ramopel_prefill_flops if label == "ramopel" else kizezen_prefill_flops)(cfg, prefill_tokens)
+            together = _prefill_together(lm, _prompts(rng, batch, prompt_tokens, vocab["vocab_size"]))
+            rec[label] = {
+                "decode_tokens_per_s": dec["value"], "decode_ms_per_step": dec["ms_per_step"], "launches_per_step": dec["launches"] / steps,
+                "decode_bytes": bytes_step, "decode_frac_of_copy": bytes_step["total"] / (dec["ms_per_step"] / 1e3) / 1e9 / pk["hbm_gbs"],
+                "prefill_tokens_per_s": pre["value"], "prefill_ms": pre["ms"], "prefill_flops": flops,
+                "prefill_batch_tokens_per_s": together["value"], "prefill_batch_ms": together["ms"],
+                "prefill_frac_of_gemm": flops / (pre["ms"] / 1e3) / (pk["bf16_tflops"] * 1e12) if dtype == "bfloat16" else None,
+                "clocks": dec["clocks"]}
+            del lm
+            torch.cuda.empty_cache()
+        out["sizes"][size] = rec
+    return out
+
+
 def ablate_decode(batch: int = 8, prompt_tokens: int = 2048, dtype: str = "bfloat16", layers: int | None = None,
                   config_index: int = 2, reps: int = 50) -> dict:
     """Where a decode step's time goes: the captured step graph is timed whole, and again with

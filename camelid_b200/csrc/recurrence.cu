@@ -734,8 +734,9 @@ __global__ void __launch_bounds__(128) general_delta_kernel(const GeneralDelta p
                 S[i + 2] = fmaf(kr[i + 2], fmaf(av.z, rem, vcol), wv.z * S[i + 2]);
                 S[i + 3] = fmaf(kr[i + 3], fmaf(av.w, rem, vcol), wv.w * S[i + 3]);
             }
+            // (a plain store might alias the buffers in shared memory as far as the compiler knows, and hold back the next token's loads)
             if (live && slice == 0)
-                p.out[((size_t)(row0 + t0 + t) * heads + hd) * Dv + c] = fmaf(sc.z, vcol, fmaf(-sc.y, pk, qr));
+                asm volatile("st.global.f32 [%0], %1;" ::"l"(p.out + ((size_t)(row0 + t0 + t) * heads + hd) * Dv + c), "f"(fmaf(sc.z, vcol, fmaf(-sc.y, pk, qr))));
         };
         const int nt = min(GD_TOKENS, n - t0);
         if (nt == GD_TOKENS) {                             // a whole round unrolled: the next tokens' loads and this one's read-out overlap

@@ -95,29 +95,32 @@ def delta_decays(h, t):
     return np.exp(-DECAY_RATE * sigmoid(np.tanh(h @ t["w1"].T) @ t["w2"].T + t["w0"]))
 
 
-def delta_core(r, k, v, w, a, heads):
-    """[n, H, D]: the read-outs S_t^T r_t token by token from S = 0; every argument [n, H * D]."""
+def delta_core(r, k, v, w, a, heads, conditioning=None):
+    """[n, H, Dv]: the read-outs S_t^T r_t token by token from S = 0; r, k, w, a [n, H * D], v [n, H * Dv]. `conditioning`
+    (a list) gets, per row, the smallest ratio over the heads of |o_t| to |r_t| |S_t|: where it is tiny the read-out is
+    what cancellation left, and the norm behind it, which keeps only the direction, magnifies whatever rounding the
+    terms carry."""
     n = r.shape[0]
     r, k, v, w, a = (np.asarray(x, dtype=np.float64).reshape(n, heads, -1) for x in (r, k, v, w, a))
     D, Dv = k.shape[-1], v.shape[-1]
-    out = np.zeros((n, heads, Dv))
+    out, ratio = np.zeros((n, heads, Dv)), np.full(n, np.inf)
     for hd in range(heads):
         S = np.zeros((D, Dv))
         for i in range(n):
             u = k[i, hd] / np.sqrt(np.sum(k[i, hd] ** 2) + 1e-6)
             S = w[i, hd][:, None] * S - np.outer(a[i, hd] * u, u @ S) + np.outer(k[i, hd], v[i, hd])
             out[i, hd] = S.T @ r[i, hd]
+            ratio[i] = min(ratio[i], np.linalg.norm(out[i, hd]) / (np.linalg.norm(r[i, hd]) * np.linalg.norm(S)))
+    if conditioning is not None:
+        conditioning.append(ratio)
     return out
 
 
-def general_delta_mixer(h, t, m, eps, sizes=None):
+def general_delta_mixer(h, t, m, eps, conditioning=None):
     n = h.shape[0]
     r, k, v = h @ t["r"].T, h @ t["k"].T, h @ t["v"].T
     w, a = delta_decays(h, t), sigmoid(h @ t["a"].T + t["a.b"])
-    o = delta_core(r, k, v, w, a, m["heads"])
-    if sizes is not None:          # per row: the smallest |o| over the heads against |r| times the norm of the current write
-        nr = lambda x: np.linalg.norm(x.reshape(n, m["heads"], -1), axis=-1)        # noqa: E731
-        sizes.append(np.min(np.linalg.norm(o, axis=-1) / (nr(r) * nr(k) * nr(v)), axis=-1))
+    o = delta_core(r, k, v, w, a, m["heads"], conditioning)
     return (rms_norm(o, None, eps).reshape(n, -1) * t["norm"] * sigmoid(h @ t["g"].T)) @ t["o"].T
 
 
@@ -168,9 +171,9 @@ def part(tensors, prefix):
     return {k[len(prefix):]: np.asarray(v, dtype=np.float64) for k, v in tensors.items() if k.startswith(prefix)}
 
 
-def forward(cfg, tensors, tokens, layers_out=None, gaps=None, sizes=None):
+def forward(cfg, tensors, tokens, layers_out=None, gaps=None, conditioning=None):
     """Logits [tokens, vocab] of one sequence; `layers_out` (a list) gets the stream after every layer, `gaps` one array
-    per routed layer (see `moe_ff`), `sizes` one per delta-rule layer."""
+    per routed layer (see `moe_ff`), `conditioning` one per delta-rule layer (see `delta_core`)."""
     eps = cfg["norm"]["eps"]
     T = {k: np.asarray(v, dtype=np.float64) for k, v in tensors.items()}
     x = T["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
@@ -184,7 +187,7 @@ def forward(cfg, tensors, tokens, layers_out=None, gaps=None, sizes=None):
                 kept[i] = latent_rows(h @ t["dkv"].T, t, m, eps)
             y = latent_attention_mixer(h, t, m, eps, kept[i if m.get("kv_from") is None else m["kv_from"]])
         else:
-            y = general_delta_mixer(h, t, m, eps, sizes)
+            y = general_delta_mixer(h, t, m, eps, conditioning)
         if mlp:
             h2, tf = zero_centred_norm(x, T[p + "norm2"], eps), part(T, p + "mlp.")
             y = y + (dense_ff(h2, tf, eps) if mlp["kind"] == "dense" else moe_ff(h2, tf, mlp, gaps))
