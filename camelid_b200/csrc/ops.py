@@ -129,6 +129,10 @@ _SIGNATURES = {
                                            c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
     ("recurrence", "cml_delta_inputs"): [c_void_p, c_long, c_int, c_long, c_void_p, c_int, c_long, c_void_p, c_int, c_int, c_void_p,
                                          c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    ("recurrence", "cml_delta_chunks"): [c_void_p, c_long, c_int, c_long, c_void_p, c_int, c_long, c_void_p, c_void_p, c_float, c_void_p,
+                                         c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    ("recurrence", "cml_delta_chunk_scan"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                             c_int, c_void_p],
     ("recurrence", "cml_general_delta_scan"): [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                                c_int, c_int, c_int, c_int, c_void_p],
     ("attention_window", "cml_qk_norm_kv_write"): [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p,
@@ -791,6 +795,51 @@ def general_delta_scan(packed: torch.Tensor, scal: torch.Tensor, state: torch.Te
     _check(_fn("recurrence", "cml_general_delta_scan")(_p(packed), _p(scal), _p(state), _p(seq_row0), _p(seq_new), _p(seq_start),
                                                        _p(seq_slot), _p(out), n_seqs, heads, key_dim, value_dim, _stream()),
            "general_delta_scan")
+
+
+DELTA_CHUNK = 16               # tokens of a chunk of the delta rule's chunked form; GDC in recurrence.cu
+
+
+def delta_chunk_floats(key_dim: int, value_dim: int) -> int:
+    """Floats ``delta_chunks`` leaves per (chunk, head)."""
+    return (4 * DELTA_CHUNK + 1) * key_dim + DELTA_CHUNK * DELTA_CHUNK + DELTA_CHUNK * value_dim
+
+
+def delta_chunks_usable(key_dim: int, value_dim: int, rate: float = 1.0) -> bool:
+    """Sizes in whole 16-byte pieces, and decays that a chunk's product can take in float32 (at least exp(-2))."""
+    return 4 <= key_dim <= 256 and key_dim % 4 == 0 and value_dim % 4 == 0 and 0.0 <= rate <= 2.0
+
+
+def delta_chunks(proj: torch.Tensor, high: torch.Tensor, a_bias: torch.Tensor, w0: torch.Tensor, rate: float, tile_seq, tile_q0,
+                 n_tiles: int, seq_row0, seq_new, chunks: torch.Tensor, heads: int, key_dim: int, value_dim: int, gate_out=None):
+    """The generalized delta rule's chunked form, first half: everything that does not depend on the state, for every chunk of
+    16 tokens (``tile_seq`` / ``tile_q0``: the step's tiles of 16 rows) and head. ``proj`` and ``gate_out`` as in ``delta_inputs``,
+    ``high`` the decays' inputs (float32 rows or split sums); ``chunks`` float32 [tiles, heads, ``delta_chunk_floats``]."""
+    _dev(proj, high, a_bias, w0, tile_seq, tile_q0, seq_row0, seq_new, chunks, gate_out)
+    proj = proj.unsqueeze(0) if proj.dim() == 2 else proj
+    high = high.unsqueeze(0) if high.dim() == 2 else high
+    rows, hd, hv = proj.shape[1], heads * key_dim, heads * value_dim
+    assert delta_chunks_usable(key_dim, value_dim) and proj.dtype == torch.float32 and proj.stride(2) == 1 and proj.shape[2] >= 3 * hd + 2 * hv
+    assert high.dtype == torch.float32 and high.shape[1:] == (rows, hd) and high.stride(2) == 1 and high.stride(1) == hd
+    assert a_bias.dtype == w0.dtype == torch.float32 and a_bias.numel() == hd == w0.numel()
+    assert chunks.dtype == torch.float32 and chunks.is_contiguous() and chunks.shape == (n_tiles, heads, delta_chunk_floats(key_dim, value_dim))
+    assert gate_out is None or (gate_out.dtype == torch.float32 and gate_out.is_contiguous() and gate_out.shape == (rows, hv))
+    _check(_fn("recurrence", "cml_delta_chunks")(
+        _p(proj), proj.stride(1), proj.shape[0], proj.stride(0), _p(high), high.shape[0], high.stride(0), _p(a_bias), _p(w0), float(rate),
+        _p(tile_seq), _p(tile_q0), int(n_tiles), _p(seq_row0), _p(seq_new), _p(chunks), _p(gate_out), heads, key_dim, value_dim, _stream()),
+        "delta_chunks")
+
+
+def delta_chunk_scan(chunks: torch.Tensor, state: torch.Tensor, seq_row0, seq_new, seq_start, seq_slot, out: torch.Tensor, n_seqs: int,
+                     heads: int, key_dim: int, value_dim: int):
+    """The second half: every sequence's chunks (in the order of its tiles) walked with its state, ``state`` and ``out`` as in
+    ``general_delta_scan``."""
+    _dev(chunks, state, seq_row0, seq_new, seq_start, seq_slot, out)
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (chunks, state, out))
+    assert chunks.shape[1:] == (heads, delta_chunk_floats(key_dim, value_dim)) and state.shape[1:] == (heads, value_dim, key_dim)
+    assert out.shape[1] == heads * value_dim
+    _check(_fn("recurrence", "cml_delta_chunk_scan")(_p(chunks), _p(state), _p(seq_row0), _p(seq_new), _p(seq_start), _p(seq_slot),
+                                                     _p(out), n_seqs, heads, key_dim, value_dim, _stream()), "delta_chunk_scan")
 
 
 def rotate_rows_(x: torch.Tensor, col0: int, heads: int, head_dim: int, rotary_dim: int, interleaved: bool, inv_freq, amp: float,

@@ -783,6 +783,355 @@ extern "C" int cml_general_delta_scan(const float* packed, const float* scal, fl
 }
 
 // ------------------------------------------------------------------------------------
+// The generalized delta rule by chunks of GDC = 16 tokens, for steps that bring several tokens per sequence. With
+// W_t the product of the decays of the chunk's tokens up to t (per key channel; W_0 = 1) and S_t = diag(W_t) Z_t the rule is
+//
+//   Z_t = Z_(t-1) - al_t (be_t^T Z_(t-1)) + ka_t v_t^T,     al = a * u / W_t,  be = u * W_(t-1),  ka = k / W_t,  rh = r * W_t
+//
+// so with M = be al^T, N = be ka^T (strictly lower triangles), Qa = rh al^T, Qk = rh ka^T (with the diagonal), S the state
+// before the chunk and P = be^T Z row by row:
+//
+//   (I + M) P = be S + N V     =>  P = B' S + N' V,    B' = (I + M)^-1 be,  N' = (I + M)^-1 N
+//   O = rh S + Qk V - Qa P     =  R' S + E V,          R' = rh - Qa B',     E = Qk - Qa N'
+//   S <- diag(W) (S + ka^T V - al^T P) = diag(W) S + G^T V - A'^T (B' S),   A' = al * W,  G = (ka - N'^T al) * W
+//
+// Everything but the three products with S and V is made by the first kernel for all chunks side by side; the
+// second walks a sequence's chunks with the state in registers. All in float: a decay is at least exp(-rate), so W stays
+// above exp(-16 rate), and every al, ka meets the be, rh of a later token, so no product grows.
+#define GDC 16
+#define GDC_FLOATS(D, Dv) ((size_t)(4 * GDC + 1) * (D) + GDC * GDC + GDC * (Dv))      // B', R', G, A', W, E, V of a (chunk, head)
+
+struct DeltaChunks {
+    const float* proj; long ld; int n_splits; long split_stride;
+    const float* high; int n_high; long high_stride;
+    const float* a_bias; const float* w0;
+    float rate;
+    const int* tile_seq; const int* tile_q0; const int* seq_row0; const int* seq_new;
+    float* chunks; float* gate_out;
+    int heads, D, Dv;
+};
+
+__global__ void __launch_bounds__(256) delta_chunks_kernel(const DeltaChunks p) {
+    extern __shared__ __align__(16) float dc_sh[];
+    __shared__ float sM[GDC][GDC + 1], sN[GDC][GDC + 1], sQk[GDC][GDC + 1], sQa[GDC][GDC + 1], s_inv[GDC];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int tile = blockIdx.x, hd = blockIdx.y, D = p.D, Dv = p.Dv, HD = p.heads * D, HV = p.heads * Dv;
+    const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile];
+    const int nt = min(GDC, p.seq_new[seq] - q0), row0 = p.seq_row0[seq] + q0;
+    const int pitch = D + 4, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    float* be = dc_sh;
+    float* al = be + GDC * pitch;
+    float* ka = al + GDC * pitch;
+    float* rh = ka + GDC * pitch;
+    float* out = p.chunks + ((size_t)tile * p.heads + hd) * GDC_FLOATS(D, Dv);
+    const int d = tid, c = hd * D + d;
+    if (d < D) {
+#pragma unroll
+        for (int t = 0; t < GDC; ++t)
+            ka[t * pitch + d] = t < nt ? split_sum(p.proj + (size_t)(row0 + t) * p.ld + HD + c, p.n_splits, p.split_stride) : 0.f;
+    }
+    __syncthreads();
+    for (int t = warp; t < GDC; t += 8) {
+        float ss = 0.f;
+        for (int i = lane; i < D; i += 32) ss = fmaf(ka[t * pitch + i], ka[t * pitch + i], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) s_inv[t] = 1.0f / sqrtf(ss + 1e-6f);
+    }
+    __syncthreads();
+    float W = 1.0f;
+    if (d < D) {
+        const float ab = p.a_bias[c], w0 = p.w0[c];
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            const bool there = t < nt;
+            const float* row = p.proj + (size_t)(row0 + (there ? t : 0)) * p.ld;
+            const float r = split_sum(row + c, p.n_splits, p.split_stride);
+            const float a = sigmoid_f(split_sum(row + 2 * HD + HV + c, p.n_splits, p.split_stride) + ab);
+            const float z = split_sum(p.high + (size_t)(row0 + (there ? t : 0)) * HD + c, p.n_high, p.high_stride) + w0;
+            const float w = there ? expf(-p.rate * sigmoid_f(z)) : 1.0f;      // tokens that are not there change nothing
+            const float k = ka[t * pitch + d], u = k * s_inv[t];
+            be[t * pitch + d] = u * W;
+            W *= w;
+            const float inv = 1.0f / W;
+            al[t * pitch + d] = there ? a * u * inv : 0.f;
+            ka[t * pitch + d] = k * inv;
+            rh[t * pitch + d] = there ? r * W : 0.f;
+        }
+        out[4 * GDC * D + d] = W;
+    }
+    for (int i = tid; i < GDC * Dv; i += 256) {            // the values, and the gate's inputs
+        const int t = i / Dv, e = i - t * Dv;
+        const float* row = p.proj + (size_t)(row0 + (t < nt ? t : 0)) * p.ld;
+        const float v = split_sum(row + 2 * HD + hd * Dv + e, p.n_splits, p.split_stride);
+        out[(4 * GDC + 1) * D + GDC * GDC + i] = t < nt ? v : 0.f;
+        if (p.gate_out && t < nt)
+            p.gate_out[(size_t)(row0 + t) * HV + hd * Dv + e] = split_sum(row + 3 * HD + HV + hd * Dv + e, p.n_splits, p.split_stride);
+    }
+    __syncthreads();
+    {   // thread (t, j), j <= t: the four products of its pair of tokens
+        const int t = tid >> 4, j = tid & 15;
+        float m = 0.f, n = 0.f, qk = 0.f, qa = 0.f;
+        if (j <= t) {
+            for (int i = 0; i < D; i += 4) {
+                const float4 b = *reinterpret_cast<const float4*>(be + t * pitch + i), r = *reinterpret_cast<const float4*>(rh + t * pitch + i);
+                const float4 a = *reinterpret_cast<const float4*>(al + j * pitch + i), k = *reinterpret_cast<const float4*>(ka + j * pitch + i);
+                m = fmaf(b.x, a.x, fmaf(b.y, a.y, fmaf(b.z, a.z, fmaf(b.w, a.w, m))));
+                n = fmaf(b.x, k.x, fmaf(b.y, k.y, fmaf(b.z, k.z, fmaf(b.w, k.w, n))));
+                qk = fmaf(r.x, k.x, fmaf(r.y, k.y, fmaf(r.z, k.z, fmaf(r.w, k.w, qk))));
+                qa = fmaf(r.x, a.x, fmaf(r.y, a.y, fmaf(r.z, a.z, fmaf(r.w, a.w, qa))));
+            }
+        }
+        sM[t][j] = j < t ? m : 0.f;
+        sN[t][j] = j < t ? n : 0.f;
+        sQk[t][j] = qk;
+        sQa[t][j] = qa;
+    }
+    __syncthreads();
+    float x[GDC];
+    if (tid < GDC) {                                       // N' by columns, in place
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            float v = sN[t][tid];
+#pragma unroll
+            for (int j = 0; j < t; ++j) v = fmaf(-sM[t][j], x[j], v);
+            x[t] = v;
+        }
+        __syncwarp(0xffff);
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) sN[t][tid] = x[t];
+    }
+    if (d < D) {                                           // B' by columns, then R'
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            float v = be[t * pitch + d];
+#pragma unroll
+            for (int j = 0; j < t; ++j) v = fmaf(-sM[t][j], x[j], v);
+            x[t] = v;
+            out[t * D + d] = v;
+        }
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            float v = rh[t * pitch + d];
+#pragma unroll
+            for (int j = 0; j <= t; ++j) v = fmaf(-sQa[t][j], x[j], v);
+            out[(GDC + t) * D + d] = v;
+        }
+    }
+    __syncthreads();                                       // N' is complete
+    if (d < D) {
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) x[t] = al[t * pitch + d];
+#pragma unroll
+        for (int j = 0; j < GDC; ++j) {
+            float v = ka[j * pitch + d];
+#pragma unroll
+            for (int t = j + 1; t < GDC; ++t) v = fmaf(-sN[t][j], x[t], v);
+            out[(2 * GDC + j) * D + d] = v * W;
+            out[(3 * GDC + j) * D + d] = x[j] * W;
+        }
+    }
+    {
+        const int t = tid >> 4, j = tid & 15;
+        float v = sQk[t][j];
+        for (int i = j + 1; i <= t; ++i) v = fmaf(-sQa[t][i], sN[i][j], v);
+        out[(4 * GDC + 1) * D + tid] = j <= t ? v : 0.f;
+    }
+}
+
+extern "C" int cml_delta_chunks(const float* proj, long ld, int n_splits, long split_stride, const float* high, int n_high,
+                                long high_stride, const float* a_bias, const float* w0, float rate, const int* tile_seq,
+                                const int* tile_q0, int n_tiles, const int* seq_row0, const int* seq_new, float* chunks,
+                                float* gate_out, int heads, int D, int Dv, void* stream) {
+    if (n_tiles <= 0) return 0;
+    if (heads < 1 || heads > 65535 || D < 4 || D > 256 || (D & 3) || Dv < 4 || (Dv & 3) || n_splits < 1 || n_high < 1 || rate < 0.f || rate > 2.f)
+        return CML_ERR_BAD_SIZE;
+    DeltaChunks p = {proj, ld, n_splits, split_stride, high, n_high, high_stride, a_bias, w0, rate, tile_seq, tile_q0, seq_row0, seq_new,
+                     chunks, gate_out, heads, D, Dv};
+    const size_t smem = (size_t)4 * GDC * (D + 4) * sizeof(float);
+    if (smem > 48 * 1024 && cml_allow_smem<delta_chunks_kernel>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE;
+    launch_pdl(delta_chunks_kernel, dim3(n_tiles, heads), dim3(256), smem, (cudaStream_t)stream, p);
+    return cml_launch_status();
+}
+
+// The walk over a sequence's chunks. A warp owns COLS columns of the state of one (sequence, head): NS lanes of DS key
+// channels each hold CPT columns, and 32 / NS such groups stand side by side. The products with the state give every lane
+// partial sums over its channels for 32 / CPT rows at a time; they are added over the lanes by halving (each step
+// hands half of the values over, so a lane ends with sums of its own), in a fixed order. The chunk's matrices come by
+// cp.async into one of two buffers while the other one's chunk is worked on.
+struct ChunkScan {
+    const float* chunks; float* state;
+    const int* seq_new; const int* seq_row0; const int* seq_start; const int* seq_slot;
+    float* out;
+    int heads, D, Dv;
+};
+
+template <int DS, int NS, int CPT, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) delta_chunk_scan_kernel(const ChunkScan p) {
+    constexpr int G = 32 / NS, WCOLS = G * CPT, COLS = WARPS * WCOLS;
+    constexpr int RG = NS / CPT;                           // rows of a group: its RG x CPT sums end in its NS lanes
+    constexpr int DP = NS * DS;
+    constexpr int THREADS = WARPS * 32;
+    extern __shared__ __align__(16) float cs_sh[];
+    const int D = p.D, Dv = p.Dv, heads = p.heads;
+    constexpr int BUF = (4 * GDC + 1) * DP + GDC * GDC + GDC * COLS;
+    float* sP = cs_sh + 2 * BUF;                           // [GDC][COLS]: B' S
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, hd = blockIdx.y, col0 = blockIdx.z * COLS;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int group = lane / NS, slice = lane % NS, d0 = slice * DS;
+    const int n = p.seq_new[s], row0 = p.seq_row0[s];
+    const bool fresh = p.seq_start[s] == 0;
+    int first = 0;                                         // chunks of the sequences before this one
+    for (int q = 0; q < s; ++q) first += (p.seq_new[q] + GDC - 1) / GDC;
+    const int n_chunks = (n + GDC - 1) / GDC;
+    const int wc = warp * WCOLS + group * CPT;             // this lane's first column within the block
+    float S[CPT][DS];
+    size_t cell[CPT];
+    bool live[CPT];
+#pragma unroll
+    for (int e = 0; e < CPT; ++e) {
+        live[e] = col0 + wc + e < Dv && d0 < D;
+        cell[e] = (((size_t)p.seq_slot[s] * heads + hd) * Dv + (col0 + wc + e < Dv ? col0 + wc + e : 0)) * D + (d0 < D ? d0 : 0);
+#pragma unroll
+        for (int i = 0; i < DS; i += 4) {
+            const bool ok = live[e] && d0 + i < D && !fresh;
+            const float4 t = *reinterpret_cast<const float4*>(p.state + cell[e] + (ok ? i : 0));
+            S[e][i] = ok ? t.x : 0.f; S[e][i + 1] = ok ? t.y : 0.f; S[e][i + 2] = ok ? t.z : 0.f; S[e][i + 3] = ok ? t.w : 0.f;
+        }
+    }
+    if (D < DP || Dv - col0 < COLS) {                      // channels and columns that are not there stay zero
+        for (int i = tid; i < 2 * BUF; i += THREADS) cs_sh[i] = 0.f;
+        __syncthreads();
+    }
+    auto fetch = [&](int ch, int buf) {
+        const float* src = p.chunks + ((size_t)(first + ch) * heads + hd) * GDC_FLOATS(D, Dv);
+        float* dst = cs_sh + buf * BUF;
+        if (D == DP) {                                     // all matrices and E in one run of memory
+            for (int i = tid * 4; i < (4 * GDC + 1) * DP + GDC * GDC; i += THREADS * 4) gd_copy<16>(dst + i, src + i);
+        } else {
+            for (int r = warp; r < 4 * GDC + 1; r += WARPS)
+                for (int i = lane * 4; i < D; i += 128) gd_copy<16>(dst + r * DP + i, src + (size_t)r * D + i);
+            for (int i = tid * 4; i < GDC * GDC; i += THREADS * 4) gd_copy<16>(dst + (4 * GDC + 1) * DP + i, src + (size_t)(4 * GDC + 1) * D + i);
+        }
+        const float* v = src + (size_t)(4 * GDC + 1) * D + GDC * GDC + col0;
+        for (int i = tid; i < GDC * COLS / 4; i += THREADS) {
+            const int t = i / (COLS / 4), e = (i % (COLS / 4)) * 4;
+            if (col0 + e < Dv) gd_copy<16>(dst + (4 * GDC + 1) * DP + GDC * GDC + t * COLS + e, v + (size_t)t * Dv + e);
+        }
+    };
+    fetch(0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    for (int ch = 0; ch < n_chunks; ++ch) {
+        if (ch + 1 < n_chunks) fetch(ch + 1, (ch + 1) & 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");       // all but the newest group: this chunk is here
+        __syncthreads();
+        const float* m = cs_sh + (ch & 1) * BUF;
+        const float* sE = m + (4 * GDC + 1) * DP;
+        const float* sV = sE + GDC * GDC;
+        const int nt = min(GDC, n - ch * GDC);
+        // B' S and R' S, RG rows at a time
+#pragma unroll
+        for (int rg = 0; rg < 2 * GDC; rg += RG) {
+            float acc[NS];                                 // value r * CPT + e: row rg + r, column e
+#pragma unroll
+            for (int r = 0; r < RG; ++r) {
+#pragma unroll
+                for (int e = 0; e < CPT; ++e) acc[r * CPT + e] = 0.f;
+#pragma unroll
+                for (int i = 0; i < DS; i += 4) {
+                    const float4 b = *reinterpret_cast<const float4*>(m + (rg + r) * DP + d0 + i);
+#pragma unroll
+                    for (int e = 0; e < CPT; ++e)
+                        acc[r * CPT + e] = fmaf(b.x, S[e][i], fmaf(b.y, S[e][i + 1], fmaf(b.z, S[e][i + 2], fmaf(b.w, S[e][i + 3], acc[r * CPT + e]))));
+                }
+            }
+#pragma unroll
+            for (int h = NS / 2; h > 0; h >>= 1) {         // lane bit h keeps the upper half of what is left
+                const bool up = (slice & h) != 0;
+#pragma unroll
+                for (int i = 0; i < h; ++i) {
+                    const float give = up ? acc[i] : acc[i + h], keep = up ? acc[i + h] : acc[i];
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+                }
+            }
+            const int row = rg + slice / CPT, e = slice % CPT;     // the sum this lane ended with
+            if (row < GDC) {
+                sP[row * COLS + wc + e] = acc[0];
+            } else {
+                const int t = row - GDC;
+                float o = acc[0];
+#pragma unroll
+                for (int j = 0; j < GDC; j += 4) {
+                    const float4 w = *reinterpret_cast<const float4*>(sE + t * GDC + j);
+                    o = fmaf(w.x, sV[j * COLS + wc + e], o);
+                    o = fmaf(w.y, sV[(j + 1) * COLS + wc + e], o);
+                    o = fmaf(w.z, sV[(j + 2) * COLS + wc + e], o);
+                    o = fmaf(w.w, sV[(j + 3) * COLS + wc + e], o);
+                }
+                if (t < nt && col0 + wc + e < Dv)
+                    asm volatile("st.global.f32 [%0], %1;" ::"l"(p.out + ((size_t)(row0 + ch * GDC + t) * heads + hd) * Dv + col0 + wc + e), "f"(o));
+            }
+        }
+        __syncwarp();                                      // a warp reads back its own columns of sP
+        // S <- diag(W) S + G^T V - A'^T (B' S)
+#pragma unroll
+        for (int i = 0; i < DS; i += 4) {
+            const float4 w = *reinterpret_cast<const float4*>(m + 4 * GDC * DP + d0 + i);
+#pragma unroll
+            for (int e = 0; e < CPT; ++e) { S[e][i] *= w.x; S[e][i + 1] *= w.y; S[e][i + 2] *= w.z; S[e][i + 3] *= w.w; }
+        }
+#pragma unroll
+        for (int j = 0; j < GDC; ++j) {
+            float v[CPT], q[CPT];
+#pragma unroll
+            for (int e = 0; e < CPT; ++e) { v[e] = sV[j * COLS + wc + e]; q[e] = -sP[j * COLS + wc + e]; }
+#pragma unroll
+            for (int i = 0; i < DS; i += 4) {
+                const float4 g = *reinterpret_cast<const float4*>(m + (2 * GDC + j) * DP + d0 + i), a = *reinterpret_cast<const float4*>(m + (3 * GDC + j) * DP + d0 + i);
+#pragma unroll
+                for (int e = 0; e < CPT; ++e) {
+                    S[e][i] = fmaf(g.x, v[e], fmaf(a.x, q[e], S[e][i]));
+                    S[e][i + 1] = fmaf(g.y, v[e], fmaf(a.y, q[e], S[e][i + 1]));
+                    S[e][i + 2] = fmaf(g.z, v[e], fmaf(a.z, q[e], S[e][i + 2]));
+                    S[e][i + 3] = fmaf(g.w, v[e], fmaf(a.w, q[e], S[e][i + 3]));
+                }
+            }
+        }
+        __syncthreads();                                   // before the next fetch overwrites this buffer
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int e = 0; e < CPT; ++e)
+#pragma unroll
+        for (int i = 0; i < DS; i += 4)
+            if (live[e] && d0 + i < D)
+                *reinterpret_cast<float4*>(p.state + cell[e] + i) = make_float4(S[e][i], S[e][i + 1], S[e][i + 2], S[e][i + 3]);
+}
+
+extern "C" int cml_delta_chunk_scan(const float* chunks, float* state, const int* seq_row0, const int* seq_new, const int* seq_start,
+                                    const int* seq_slot, float* out, int n_seqs, int heads, int D, int Dv, void* stream) {
+    if (n_seqs <= 0) return 0;
+    if (heads < 1 || heads > 65535 || D < 4 || D > 256 || (D & 3) || Dv < 4 || (Dv & 3)) return CML_ERR_BAD_SIZE;
+    if ((((uintptr_t)chunks) | ((uintptr_t)state)) & 15) return CML_ERR_BAD_ALIGN;
+    ChunkScan p = {chunks, state, seq_new, seq_row0, seq_start, seq_slot, out, heads, D, Dv};
+#define CS_CASE(DS_, NS_, CPT_, WARPS_)                                                                                            \
+    if (D <= NS_ * DS_) {                                                                                                          \
+        constexpr int COLS = WARPS_ * (32 / NS_) * CPT_;                                                                           \
+        constexpr size_t smem = (size_t)(2 * ((4 * GDC + 1) * NS_ * DS_ + GDC * GDC + GDC * COLS) + GDC * COLS) * sizeof(float);   \
+        if (smem > 48 * 1024 && cml_allow_smem<delta_chunk_scan_kernel<DS_, NS_, CPT_, WARPS_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE; \
+        launch_pdl(delta_chunk_scan_kernel<DS_, NS_, CPT_, WARPS_>, dim3(n_seqs, heads, (Dv + COLS - 1) / COLS), dim3(WARPS_ * 32), smem, \
+                   (cudaStream_t)stream, p);                                                                                       \
+        return cml_launch_status();                                                                                                \
+    }
+    CS_CASE(4, 8, 2, 2) CS_CASE(4, 16, 2, 4) CS_CASE(4, 32, 4, 4) CS_CASE(8, 32, 4, 4)
+#undef CS_CASE
+    return CML_ERR_BAD_SIZE;
+}
+
+// ------------------------------------------------------------------------------------
 // Rotation of heads inside float rows, in place: x [rows, ld] holds `heads` heads of D channels from column col0; the
 // first rot_dim channels of every head are turned by angle = position * inv_freq[i] (pairing 1: channels (2i, 2i + 1);
 // 0: channels (i, i + rot_dim / 2)), sines and cosines times `amp`; then heads from number `scaled_from` on are

@@ -362,11 +362,12 @@ class GeneralDelta(Part):
     def cache_spec(self):
         return StateSpec((self.num_heads, self.value_dim, self.key_dim), "float32", "delta")
 
+    def query_tile_sizes(self):
+        return [ops.DELTA_CHUNK]
+
     def read_out(self, ctx, x, out=None):
         n, H, D, V = ctx.n_rows, self.num_heads, self.key_dim, self.value_dim
         sums = linear.product_f32(ctx, x, self.w_in, "gd_proj")            # split sums where the step is small: added below
-        packed = ctx.buffer("gd_packed", (n, H, 4 * D + V), torch.float32)
-        scal = ctx.buffer("gd_scalars", (n, H, 4), torch.float32)
         split = sums.dim() == 3
         gate, gate_col, high = sums, self.gate_col, None
         if split:
@@ -375,11 +376,21 @@ class GeneralDelta(Part):
             low = ctx.buffer("gd_low", (n, self.w2.shape[1]))
             ops.tanh_columns(sums, self.narrow_col, low)
             high = linear.product_f32(ctx, low, self.w2, "gd_high")
-        ops.delta_inputs(sums, self.a_bias, self.w0, self.decay_rate, packed, scal, H, D, V, high, None if high is not None else self.w2,
-                         gate if split else None)
         raw = ctx.buffer("gd_raw", (n, self.v_width), torch.float32)
-        ops.general_delta_scan(packed, scal, ctx.state("delta"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, raw,
-                               ctx.n_seqs, H, D, V)
+        if high is not None and ctx.max_new >= ops.DELTA_CHUNK and ops.delta_chunks_usable(D, V, self.decay_rate):
+            # prompts: chunks of 16 tokens side by side, then a walk over the chunks
+            tile_seq, tile_q0, n_tiles = ctx.query_tiles(ops.DELTA_CHUNK)
+            chunks = ctx.buffer("gd_chunks", (n_tiles, H, ops.delta_chunk_floats(D, V)), torch.float32)
+            ops.delta_chunks(sums, high, self.a_bias, self.w0, self.decay_rate, tile_seq, tile_q0, n_tiles, ctx.seq_row0, ctx.seq_new,
+                             chunks, H, D, V, gate if split else None)
+            ops.delta_chunk_scan(chunks, ctx.state("delta"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, raw, ctx.n_seqs, H, D, V)
+        else:
+            packed = ctx.buffer("gd_packed", (n, H, 4 * D + V), torch.float32)
+            scal = ctx.buffer("gd_scalars", (n, H, 4), torch.float32)
+            ops.delta_inputs(sums, self.a_bias, self.w0, self.decay_rate, packed, scal, H, D, V, high, None if high is not None else self.w2,
+                             gate if split else None)
+            ops.general_delta_scan(packed, scal, ctx.state("delta"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, raw,
+                                   ctx.n_seqs, H, D, V)
         if out is None:
             out = ctx.buffer("gd_out", (n, self.v_width))
         ops.head_norm_gate(raw, False, self.norm_w, True, gate, gate_col, out, H, V, self.eps)

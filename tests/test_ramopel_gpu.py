@@ -465,8 +465,9 @@ def _delta_rows(gen, T, H, D, Dv):
             "a": torch.randn(T, H * D, generator=gen) * 2, "g": torch.randn(T, H * Dv, generator=gen)}
 
 
-def _delta_scan(cuda, rows, narrow, t, rate, state, a, H, D, Dv, splits, made_here):
-    """The preparing kernel and the scan on the given rows; the projections' sums in ``splits`` shares."""
+def _delta_scan(cuda, rows, narrow, t, rate, state, a, H, D, Dv, splits, made_here, chunked=False):
+    """The preparing kernel and the scan on the given rows, token by token or by chunks of 16; the projections' sums in
+    ``splits`` shares."""
     from camelid_b200.csrc import ops
     n = rows["r"].shape[0]
     proj = torch.cat([rows[x] for x in "rkvag"] + [narrow], 1)
@@ -476,22 +477,36 @@ def _delta_scan(cuda, rows, narrow, t, rate, state, a, H, D, Dv, splits, made_he
     packed = torch.empty(n, H, 4 * D + Dv, device=cuda)
     scal = torch.empty(n, H, 4, device=cuda)
     gate = torch.empty(n, H * Dv, device=cuda)
+    out = torch.empty(n, H * Dv, device=cuda)
     high = None
-    if not made_here:
+    if chunked or not made_here:
         low = torch.empty(n, narrow.shape[1], device=cuda)
         ops.tanh_columns(proj.to(cuda), 3 * H * D + 2 * H * Dv, low)
         high = (low.double() @ t["w2"].double().to(cuda).T).float()
+    if chunked:
+        dev = lambda x: torch.tensor(x, dtype=torch.int32, device=cuda)      # noqa: E731
+        tiles = [(s, q0) for s, k in enumerate(a["seq_new"].tolist()) for q0 in range(0, k, ops.DELTA_CHUNK)]
+        chunks = torch.full((len(tiles), H, ops.delta_chunk_floats(D, Dv)), float("nan"), device=cuda)
+        ops.delta_chunks(proj.to(cuda), high, t["a.b"].to(cuda), t["w0"].to(cuda), rate, dev([x[0] for x in tiles]), dev([x[1] for x in tiles]),
+                         len(tiles), a["seq_row0"], a["seq_new"], chunks, H, D, Dv, gate)
+        ops.delta_chunk_scan(chunks, state, a["seq_row0"], a["seq_new"], a["seq_start"], a["seq_slot"], out, len(a["seq_new"]), H, D, Dv)
+        return out.cpu(), gate.cpu()
     ops.delta_inputs(proj.to(cuda), t["a.b"].to(cuda), t["w0"].to(cuda), rate, packed, scal, H, D, Dv, high, t["w2"].to(cuda) if made_here else None,
                      gate)
-    out = torch.empty(n, H * Dv, device=cuda)
     ops.general_delta_scan(packed, scal, state, a["seq_row0"], a["seq_new"], a["seq_start"], a["seq_slot"], out, len(a["seq_new"]), H, D, Dv)
     return out.cpu(), gate.cpu()
 
 
-@pytest.mark.parametrize("H,D,Dv,rank", [(3, 24, 24, 8), (1, 128, 128, 6), (2, 20, 7, 16), (2, 33, 33, 5), (1, 200, 64, 40), (4, 3, 5, 8), (2, 64, 64, 24)])
-def test_delta_rule_through_portions_and_slots(cuda, H, D, Dv, rank):
+@pytest.mark.parametrize("H,D,Dv,rank", [(3, 24, 24, 8), (1, 128, 128, 6), (2, 20, 7, 16), (2, 33, 33, 5), (1, 200, 64, 40), (4, 3, 5, 8), (2, 64, 64, 24),
+                                         (3, 28, 36, 8), (1, 256, 20, 8), (2, 100, 104, 8), (5, 4, 4, 8)])
+@pytest.mark.parametrize("chunked", [False, True])
+def test_delta_rule_through_portions_and_slots(cuda, H, D, Dv, rank, chunked):
     """Two sequences side by side in portions that differ, in slots that held other states: a key written at row 2 with
-    decays near one and removals near zero is asked for at row 140, a head that removes and decays has lost it."""
+    decays near one and removals near zero is asked for at row 140, a head that removes and decays has lost it. Token by
+    token, and by chunks of 16 (the portions end inside, at and behind a chunk's edge; single tokens in between)."""
+    from camelid_b200.csrc import ops
+    if chunked and not ops.delta_chunks_usable(D, Dv):
+        return                                                          # odd sizes are walked token by token
     gen = torch.Generator().manual_seed(6)
     T, rate = 150, float(np.exp(-0.5))
     t = {"w2": torch.randn(H * D, rank, generator=gen) * 0.3, "w0": torch.randn(H * D, generator=gen), "a.b": torch.randn(H * D, generator=gen)}
@@ -519,7 +534,8 @@ def test_delta_rule_through_portions_and_slots(cuda, H, D, Dv, rank):
         a = arrays(cuda, [at[s] for s in live], news, slots=[3 - s for s in live])
         rows = {x: torch.cat([seqs[s][0][x][at[s]:at[s] + n] for s, n in zip(live, news)]) for x in "rkvag"}
         narrow = torch.cat([seqs[s][1][at[s]:at[s] + n] for s, n in zip(live, news)])
-        out, gate = _delta_scan(cuda, rows, narrow, t, rate, state, a, H, D, Dv, 1 + step % 4, step % 2 == 0)
+        out, gate = _delta_scan(cuda, rows, narrow, t, rate, state, a, H, D, Dv, 1 + step % 4, step % 2 == 0,
+                                chunked and (max(news) > 1 or step % 2 == 0))
         assert torch.allclose(gate, rows["g"], atol=1e-5)
         r0 = 0
         for s, n in zip(live, news):
