@@ -811,9 +811,16 @@ struct DeltaChunks {
     int heads, D, Dv;
 };
 
-__global__ void __launch_bounds__(256) delta_chunks_kernel(const DeltaChunks p) {
+#define GDP 20               // floats of a row of a 16 x 16 matrix in shared memory (16-byte rows, read four at a time)
+
+// One block per (chunk, head); THREADS >= D, a thread owns a key channel. All of a thread's inputs are asked for before
+// any of them is used.
+template <int THREADS>
+__global__ void __launch_bounds__(THREADS) delta_chunks_kernel(const DeltaChunks p) {
+    constexpr int NT = 256 / THREADS;                      // pairs of tokens (t, j) of a thread
     extern __shared__ __align__(16) float dc_sh[];
-    __shared__ float sM[GDC][GDC + 1], sN[GDC][GDC + 1], sQk[GDC][GDC + 1], sQa[GDC][GDC + 1], s_inv[GDC];
+    __shared__ __align__(16) float sM[GDC][GDP], sN[GDC][GDP], sQk[GDC][GDP], sQa[GDC][GDP], sNt[GDC][GDP];
+    __shared__ float s_inv[GDC];
     pdl_wait();
     pdl_launch_dependents();
     const int tile = blockIdx.x, hd = blockIdx.y, D = p.D, Dv = p.Dv, HD = p.heads * D, HV = p.heads * Dv;
@@ -825,14 +832,49 @@ __global__ void __launch_bounds__(256) delta_chunks_kernel(const DeltaChunks p) 
     float* ka = al + GDC * pitch;
     float* rh = ka + GDC * pitch;
     float* out = p.chunks + ((size_t)tile * p.heads + hd) * GDC_FLOATS(D, Dv);
-    const int d = tid, c = hd * D + d;
-    if (d < D) {
+    const int d = min(tid, D - 1), c = hd * D + d;
+    const bool mine = tid < D;
+    float kk[GDC], rr[GDC], aa[GDC], zz[GDC];
 #pragma unroll
-        for (int t = 0; t < GDC; ++t)
-            ka[t * pitch + d] = t < nt ? split_sum(p.proj + (size_t)(row0 + t) * p.ld + HD + c, p.n_splits, p.split_stride) : 0.f;
+    for (int t = 0; t < GDC; ++t) {
+        const float* row = p.proj + (size_t)(row0 + min(t, nt - 1)) * p.ld + c;
+        kk[t] = row[HD];
+        rr[t] = row[0];
+        aa[t] = row[2 * HD + HV];
+        zz[t] = p.high[(size_t)(row0 + min(t, nt - 1)) * HD + c];
+    }
+    for (int sp = 1; sp < p.n_splits; ++sp)                // (products of few rows come as split sums)
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            const float* row = p.proj + (size_t)sp * p.split_stride + (size_t)(row0 + min(t, nt - 1)) * p.ld + c;
+            kk[t] += row[HD];
+            rr[t] += row[0];
+            aa[t] += row[2 * HD + HV];
+        }
+    for (int sp = 1; sp < p.n_high; ++sp)
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) zz[t] += p.high[(size_t)sp * p.high_stride + (size_t)(row0 + min(t, nt - 1)) * HD + c];
+    const float ab = p.a_bias[c], w0 = p.w0[c];
+    if (mine) {
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) {
+            if (t >= nt) kk[t] = 0.f;
+            ka[t * pitch + d] = kk[t];
+        }
+    }
+    for (int e = tid; e < Dv; e += THREADS) {              // the values, and the gate's inputs
+        float v[GDC];
+        const float* col = p.proj + (size_t)row0 * p.ld + 2 * HD + hd * Dv + e;
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) v[t] = split_sum(col + (size_t)min(t, nt - 1) * p.ld, p.n_splits, p.split_stride);
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) out[(4 * GDC + 1) * D + GDC * GDC + t * Dv + e] = t < nt ? v[t] : 0.f;
+        if (p.gate_out)
+            for (int t = 0; t < nt; ++t)
+                p.gate_out[(size_t)(row0 + t) * HV + hd * Dv + e] = split_sum(col + (size_t)t * p.ld + HD + HV, p.n_splits, p.split_stride);
     }
     __syncthreads();
-    for (int t = warp; t < GDC; t += 8) {
+    for (int t = warp; t < GDC; t += THREADS / 32) {
         float ss = 0.f;
         for (int i = lane; i < D; i += 32) ss = fmaf(ka[t * pitch + i], ka[t * pitch + i], ss);
         ss = warp_sum(ss);
@@ -840,102 +882,114 @@ __global__ void __launch_bounds__(256) delta_chunks_kernel(const DeltaChunks p) 
     }
     __syncthreads();
     float W = 1.0f;
-    if (d < D) {
-        const float ab = p.a_bias[c], w0 = p.w0[c];
+    if (mine) {
 #pragma unroll
         for (int t = 0; t < GDC; ++t) {
-            const bool there = t < nt;
-            const float* row = p.proj + (size_t)(row0 + (there ? t : 0)) * p.ld;
-            const float r = split_sum(row + c, p.n_splits, p.split_stride);
-            const float a = sigmoid_f(split_sum(row + 2 * HD + HV + c, p.n_splits, p.split_stride) + ab);
-            const float z = split_sum(p.high + (size_t)(row0 + (there ? t : 0)) * HD + c, p.n_high, p.high_stride) + w0;
-            const float w = there ? expf(-p.rate * sigmoid_f(z)) : 1.0f;      // tokens that are not there change nothing
-            const float k = ka[t * pitch + d], u = k * s_inv[t];
+            const bool there = t < nt;                     // tokens that are not there change nothing
+            const float w = there ? expf(-p.rate * sigmoid_f(zz[t] + w0)) : 1.0f;
+            const float u = kk[t] * s_inv[t];
             be[t * pitch + d] = u * W;
             W *= w;
             const float inv = 1.0f / W;
-            al[t * pitch + d] = there ? a * u * inv : 0.f;
-            ka[t * pitch + d] = k * inv;
-            rh[t * pitch + d] = there ? r * W : 0.f;
+            al[t * pitch + d] = there ? sigmoid_f(aa[t] + ab) * u * inv : 0.f;
+            ka[t * pitch + d] = kk[t] * inv;
+            rh[t * pitch + d] = there ? rr[t] * W : 0.f;
         }
         out[4 * GDC * D + d] = W;
     }
-    for (int i = tid; i < GDC * Dv; i += 256) {            // the values, and the gate's inputs
-        const int t = i / Dv, e = i - t * Dv;
-        const float* row = p.proj + (size_t)(row0 + (t < nt ? t : 0)) * p.ld;
-        const float v = split_sum(row + 2 * HD + hd * Dv + e, p.n_splits, p.split_stride);
-        out[(4 * GDC + 1) * D + GDC * GDC + i] = t < nt ? v : 0.f;
-        if (p.gate_out && t < nt)
-            p.gate_out[(size_t)(row0 + t) * HV + hd * Dv + e] = split_sum(row + 3 * HD + HV + hd * Dv + e, p.n_splits, p.split_stride);
-    }
     __syncthreads();
-    {   // thread (t, j), j <= t: the four products of its pair of tokens
-        const int t = tid >> 4, j = tid & 15;
-        float m = 0.f, n = 0.f, qk = 0.f, qa = 0.f;
-        if (j <= t) {
-            for (int i = 0; i < D; i += 4) {
+    {   // the four products of a pair of tokens (t, j); a thread's pairs share j
+        const int j = tid & 15;
+        float m[NT], n[NT], qk[NT], qa[NT];
+#pragma unroll
+        for (int u = 0; u < NT; ++u) m[u] = n[u] = qk[u] = qa[u] = 0.f;
+        for (int i = 0; i < D; i += 4) {
+            const float4 a = *reinterpret_cast<const float4*>(al + j * pitch + i), k = *reinterpret_cast<const float4*>(ka + j * pitch + i);
+#pragma unroll
+            for (int u = 0; u < NT; ++u) {
+                const int t = (tid >> 4) + u * (THREADS / 16);
                 const float4 b = *reinterpret_cast<const float4*>(be + t * pitch + i), r = *reinterpret_cast<const float4*>(rh + t * pitch + i);
-                const float4 a = *reinterpret_cast<const float4*>(al + j * pitch + i), k = *reinterpret_cast<const float4*>(ka + j * pitch + i);
-                m = fmaf(b.x, a.x, fmaf(b.y, a.y, fmaf(b.z, a.z, fmaf(b.w, a.w, m))));
-                n = fmaf(b.x, k.x, fmaf(b.y, k.y, fmaf(b.z, k.z, fmaf(b.w, k.w, n))));
-                qk = fmaf(r.x, k.x, fmaf(r.y, k.y, fmaf(r.z, k.z, fmaf(r.w, k.w, qk))));
-                qa = fmaf(r.x, a.x, fmaf(r.y, a.y, fmaf(r.z, a.z, fmaf(r.w, a.w, qa))));
+                m[u] = fmaf(b.x, a.x, fmaf(b.y, a.y, fmaf(b.z, a.z, fmaf(b.w, a.w, m[u]))));
+                n[u] = fmaf(b.x, k.x, fmaf(b.y, k.y, fmaf(b.z, k.z, fmaf(b.w, k.w, n[u]))));
+                qk[u] = fmaf(r.x, k.x, fmaf(r.y, k.y, fmaf(r.z, k.z, fmaf(r.w, k.w, qk[u]))));
+                qa[u] = fmaf(r.x, a.x, fmaf(r.y, a.y, fmaf(r.z, a.z, fmaf(r.w, a.w, qa[u]))));
             }
         }
-        sM[t][j] = j < t ? m : 0.f;
-        sN[t][j] = j < t ? n : 0.f;
-        sQk[t][j] = qk;
-        sQa[t][j] = qa;
+#pragma unroll
+        for (int u = 0; u < NT; ++u) {
+            const int t = (tid >> 4) + u * (THREADS / 16);
+            sM[t][j] = j < t ? m[u] : 0.f;
+            sN[t][j] = j < t ? n[u] : 0.f;
+            sQk[t][j] = j <= t ? qk[u] : 0.f;
+            sQa[t][j] = j <= t ? qa[u] : 0.f;
+        }
     }
     __syncthreads();
+    // x <- (I + M)^-1 x for a column x
+    auto solve = [&](float (&x)[GDC]) {
+#pragma unroll
+        for (int t = 1; t < GDC; ++t)
+#pragma unroll
+            for (int j = 0; j < t; j += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(&sM[t][j]);
+                x[t] = fmaf(-v.x, x[j], x[t]);
+                if (j + 1 < t) x[t] = fmaf(-v.y, x[j + 1], x[t]);
+                if (j + 2 < t) x[t] = fmaf(-v.z, x[j + 2], x[t]);
+                if (j + 3 < t) x[t] = fmaf(-v.w, x[j + 3], x[t]);
+            }
+    };
     float x[GDC];
-    if (tid < GDC) {                                       // N' by columns, in place
+    if (mine) {                                            // B', then R', column by column
 #pragma unroll
-        for (int t = 0; t < GDC; ++t) {
-            float v = sN[t][tid];
-#pragma unroll
-            for (int j = 0; j < t; ++j) v = fmaf(-sM[t][j], x[j], v);
-            x[t] = v;
-        }
-        __syncwarp(0xffff);
-#pragma unroll
-        for (int t = 0; t < GDC; ++t) sN[t][tid] = x[t];
-    }
-    if (d < D) {                                           // B' by columns, then R'
-#pragma unroll
-        for (int t = 0; t < GDC; ++t) {
-            float v = be[t * pitch + d];
-#pragma unroll
-            for (int j = 0; j < t; ++j) v = fmaf(-sM[t][j], x[j], v);
-            x[t] = v;
-            out[t * D + d] = v;
-        }
+        for (int t = 0; t < GDC; ++t) x[t] = be[t * pitch + d];
+        solve(x);
 #pragma unroll
         for (int t = 0; t < GDC; ++t) {
             float v = rh[t * pitch + d];
 #pragma unroll
-            for (int j = 0; j <= t; ++j) v = fmaf(-sQa[t][j], x[j], v);
+            for (int j = 0; j <= t; j += 4) {
+                const float4 q = *reinterpret_cast<const float4*>(&sQa[t][j]);
+                v = fmaf(-q.x, x[j], v);
+                if (j + 1 <= t) v = fmaf(-q.y, x[j + 1], v);
+                if (j + 2 <= t) v = fmaf(-q.z, x[j + 2], v);
+                if (j + 3 <= t) v = fmaf(-q.w, x[j + 3], v);
+            }
+            out[t * D + d] = x[t];
             out[(GDC + t) * D + d] = v;
         }
     }
-    __syncthreads();                                       // N' is complete
-    if (d < D) {
+    if (tid >= THREADS - 32 && lane < GDC) {               // the last warp: N' column by column, both ways round
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) x[t] = sN[t][lane];
+        solve(x);
+        __syncwarp(0xffff);
+#pragma unroll
+        for (int t = 0; t < GDC; ++t) { sN[t][lane] = x[t]; sNt[lane][t] = x[t]; }
+    }
+    __syncthreads();
+    if (mine) {
 #pragma unroll
         for (int t = 0; t < GDC; ++t) x[t] = al[t * pitch + d];
 #pragma unroll
         for (int j = 0; j < GDC; ++j) {
             float v = ka[j * pitch + d];
 #pragma unroll
-            for (int t = j + 1; t < GDC; ++t) v = fmaf(-sN[t][j], x[t], v);
+            for (int t0 = (j + 1) & ~3; t0 < GDC; t0 += 4) {
+                const float4 q = *reinterpret_cast<const float4*>(&sNt[j][t0]);
+                if (t0 > j) v = fmaf(-q.x, x[t0], v);
+                if (t0 + 1 > j) v = fmaf(-q.y, x[t0 + 1], v);
+                if (t0 + 2 > j) v = fmaf(-q.z, x[t0 + 2], v);
+                if (t0 + 3 > j) v = fmaf(-q.w, x[t0 + 3], v);
+            }
             out[(2 * GDC + j) * D + d] = v * W;
             out[(3 * GDC + j) * D + d] = x[j] * W;
         }
     }
-    {
-        const int t = tid >> 4, j = tid & 15;
+    for (int i = tid; i < GDC * GDC; i += THREADS) {
+        const int t = i >> 4, j = i & 15;
         float v = sQk[t][j];
-        for (int i = j + 1; i <= t; ++i) v = fmaf(-sQa[t][i], sN[i][j], v);
-        out[(4 * GDC + 1) * D + tid] = j <= t ? v : 0.f;
+        for (int q = j + 1; q <= t; ++q) v = fmaf(-sQa[t][q], sN[q][j], v);
+        out[(4 * GDC + 1) * D + i] = v;
     }
 }
 
@@ -949,8 +1003,12 @@ extern "C" int cml_delta_chunks(const float* proj, long ld, int n_splits, long s
     DeltaChunks p = {proj, ld, n_splits, split_stride, high, n_high, high_stride, a_bias, w0, rate, tile_seq, tile_q0, seq_row0, seq_new,
                      chunks, gate_out, heads, D, Dv};
     const size_t smem = (size_t)4 * GDC * (D + 4) * sizeof(float);
-    if (smem > 48 * 1024 && cml_allow_smem<delta_chunks_kernel>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE;
-    launch_pdl(delta_chunks_kernel, dim3(n_tiles, heads), dim3(256), smem, (cudaStream_t)stream, p);
+    if (D <= 128) {
+        launch_pdl(delta_chunks_kernel<128>, dim3(n_tiles, heads), dim3(128), smem, (cudaStream_t)stream, p);
+    } else {
+        if (smem > 32 * 1024 && cml_allow_smem<delta_chunks_kernel<256>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE;
+        launch_pdl(delta_chunks_kernel<256>, dim3(n_tiles, heads), dim3(256), smem, (cudaStream_t)stream, p);
+    }
     return cml_launch_status();
 }
 
@@ -1086,8 +1144,14 @@ __global__ void __launch_bounds__(WARPS * 32) delta_chunk_scan_kernel(const Chun
 #pragma unroll
         for (int j = 0; j < GDC; ++j) {
             float v[CPT], q[CPT];
+            if constexpr (CPT == 4) {                      // (wc is a multiple of 4)
+                const float4 vv = *reinterpret_cast<const float4*>(sV + j * COLS + wc), qq = *reinterpret_cast<const float4*>(sP + j * COLS + wc);
+                v[0] = vv.x; v[1] = vv.y; v[2] = vv.z; v[3] = vv.w;
+                q[0] = -qq.x; q[1] = -qq.y; q[2] = -qq.z; q[3] = -qq.w;
+            } else {
 #pragma unroll
-            for (int e = 0; e < CPT; ++e) { v[e] = sV[j * COLS + wc + e]; q[e] = -sP[j * COLS + wc + e]; }
+                for (int e = 0; e < CPT; ++e) { v[e] = sV[j * COLS + wc + e]; q[e] = -sP[j * COLS + wc + e]; }
+            }
 #pragma unroll
             for (int i = 0; i < DS; i += 4) {
                 const float4 g = *reinterpret_cast<const float4*>(m + (2 * GDC + j) * DP + d0 + i), a = *reinterpret_cast<const float4*>(m + (3 * GDC + j) * DP + d0 + i);
