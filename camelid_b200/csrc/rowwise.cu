@@ -306,10 +306,13 @@ rmsnorm_rows_kernel(const float* __restrict__ x, const TW* __restrict__ w, TO* _
         for (int i = 0; i < VPL; ++i) {
             const int c = (lane + 32 * i) * 4;
             if (c >= hidden) continue;
-            o[c] = from_f32<TO>(v[i].x * scale * to_f32(wt[c]));
-            o[c + 1] = from_f32<TO>(v[i].y * scale * to_f32(wt[c + 1]));
-            o[c + 2] = from_f32<TO>(v[i].z * scale * to_f32(wt[c + 2]));
-            o[c + 3] = from_f32<TO>(v[i].w * scale * to_f32(wt[c + 3]));
+            union { TO e[4]; uint2 half[sizeof(TO) / 2]; } y;          // four columns in one or two 8-byte stores
+            y.e[0] = from_f32<TO>(v[i].x * scale * to_f32(wt[c]));
+            y.e[1] = from_f32<TO>(v[i].y * scale * to_f32(wt[c + 1]));
+            y.e[2] = from_f32<TO>(v[i].z * scale * to_f32(wt[c + 2]));
+            y.e[3] = from_f32<TO>(v[i].w * scale * to_f32(wt[c + 3]));
+#pragma unroll
+            for (int k = 0; k < (int)sizeof(TO) / 2; ++k) reinterpret_cast<uint2*>(o + c)[k] = y.half[k];
         }
     };
     write(w, out + (size_t)r * hidden);
@@ -319,7 +322,7 @@ rmsnorm_rows_kernel(const float* __restrict__ x, const TW* __restrict__ w, TO* _
 template <typename TW, typename TO>
 static bool launch_rmsnorm_rows(const float* x, const void* w, void* out, const int* rows_index, int rows, int hidden,
                                 float eps, const void* w2, void* out2, cudaStream_t s) {
-    if (hidden % 4 != 0 || hidden > 4096 || rows < 64) return false;
+    if (hidden % 4 != 0 || hidden > 4096 || rows < 64 || ((((uintptr_t)out) | ((uintptr_t)out2)) & 7)) return false;
     const dim3 grid((rows + 7) / 8), block(256);
     const int vpl = (hidden / 4 + 31) / 32;
 #define CML_ROWS(V) launch_pdl(rmsnorm_rows_kernel<TW, TO, V>, grid, block, 0, s, x, (const TW*)w, (TO*)out, rows_index, rows, hidden, eps, (const TW*)w2, (TO*)out2)

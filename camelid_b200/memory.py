@@ -93,6 +93,7 @@ def plan_for_model(model, max_tokens: int = 0, max_slots: int | None = None, ste
     # widest activation in the compute type; float32 split sums of one product (up to 8 splits of
     # the rows that decode paths take, 4 of a wide step); float32 logits of one row per sequence
     per_row = 4 * hidden + e * (2 * hidden + 2 * widest + 2 * widest_kv)
+    per_row += max((p.workspace_per_row() for b in model.blocks if hasattr(b, "parts") for p in b.parts()), default=0)
     partial_rows = min(rows, 128)
     workspace = rows * per_row + 4 * 4 * rows * hidden + 8 * 4 * partial_rows * widest
     workspace += 4 * max(n_slots, 1) * model.vocab_size

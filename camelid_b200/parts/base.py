@@ -84,6 +84,11 @@ class Part:
     def cache_spec(self):
         return None
 
+    def workspace_per_row(self) -> int:
+        """Bytes of scratch a prompt step takes per row beyond what the memory plan counts for every part (activations
+        in the compute type and split sums)."""
+        return 0
+
     def query_tile_sizes(self) -> list:
         """Mixers: the sizes of query tiles (rows per tile) their prefill kernels ask the
         step context for."""

@@ -365,6 +365,11 @@ class GeneralDelta(Part):
     def query_tile_sizes(self):
         return [ops.DELTA_CHUNK]
 
+    def workspace_per_row(self):
+        # the float32 input product and decays' inputs, and the chunks' matrices
+        D, V = self.key_dim, self.value_dim
+        return 4 * (self.narrow_col + self.k_width + self.num_heads * (ops.delta_chunk_floats(D, V) // ops.DELTA_CHUNK + 1))
+
     def read_out(self, ctx, x, out=None):
         n, H, D, V = ctx.n_rows, self.num_heads, self.key_dim, self.value_dim
         sums = linear.product_f32(ctx, x, self.w_in, "gd_proj")            # split sums where the step is small: added below

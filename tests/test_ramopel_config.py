@@ -108,6 +108,15 @@ def test_refusals_name_the_key(path, value, key):
     assert key in str(e.value)
 
 
+def test_memory_plan_counts_the_chunks_scratch():
+    from camelid_b200.csrc import ops
+    model = DecoderModel.from_config(WIDE, dtype=torch.bfloat16, device="cpu")
+    part = model.blocks[1].mixer
+    assert part.workspace_per_row() >= 4 * (5 * 128 + 128 + 2 * ops.delta_chunk_floats(64, 64) // 16)
+    plan = model.memory_plan(4096, 4, 2048)
+    assert plan.workspace > 2048 * part.workspace_per_row()
+
+
 def test_missing_keys_take_their_defaults():
     cfg = copy.deepcopy(MIXED)
     del cfg["embedding"], cfg["layers"][0]["mixer"]["vdim"], cfg["layers"][0]["mixer"]["mask"], cfg["layers"][3]["mlp"]
