@@ -179,3 +179,19 @@ def test_a_mistake_in_a_mechanism_shows_in_the_logits(name, change, first):
     assert diff[:first].max(initial=0.0) == 0.0
     assert diff[first] > 1e-3 or first == 0
     assert np.median(diff[first:]) > 1e-2 and diff[first:].max() > 0.1
+
+
+def test_benchmark_counts_every_matrix_once():
+    """The bench's bytes of a decode step: with all experts reached they are the model's matrices, without the embedding
+    table; the two models of the bench pass about equally many elements per token."""
+    from camelid_b200 import benchmark as b
+    for size in b.RAMOPEL_SIZES:
+        cfg = b.ramopel_config_for(size)
+        specs = DecoderModel.from_config(cfg, dtype=torch.bfloat16, device="cpu").tensor_specs()
+        want = sum(int(np.prod(s.shape)) for n, s in specs.items() if len(s.shape) == 2 and n != "embed")
+        got = sum(b._ramopel_matrices(L, cfg["width"], L["mlp"].get("router", {}).get("experts", 0)) for L in cfg["layers"])
+        assert got + cfg["vocab"] * cfg["width"] == want
+        bytes_step = b.ramopel_step_bytes(cfg, 10 ** 4, 512.0, 2)                # so many rows reach every expert
+        assert abs(bytes_step["weights"] - 2 * want) < 1e-3 * want
+        mine, other = b.ramopel_prefill_flops(cfg, 2048), b.kizezen_prefill_flops(b.kizezen_config_like_ramopel(size), 2048)
+        assert 0.9 < mine / other < 1.1
