@@ -31,7 +31,7 @@ class LayerSpec:
     also norms every sublayer's output before it is added, x + scale * post_norm(sublayer(norm(x))),
     with ``post_norm1`` / ``post_norm2`` and ``residual_scale``. The ``postnorm`` arrangement norms the stream itself after
     every sum, x <- norm1(a x + mixer(x)), x <- norm2(a x + ffn(x)), with a = ``residual_scale``; the sublayers read x as
-    it is. ``after`` names a part (role ``layer_input``) that runs at the end of the layer and adds what it makes from the
+    it is. ``outnorm`` norms only what the sublayers hand over, x <- x + a norm1(mixer(x)), x <- x + a norm2(ffn(x)). ``after`` names a part (role ``layer_input``) that runs at the end of the layer and adds what it makes from the
     stream and the step's tokens."""
     arrangement: str
     norm1: PartSpec

@@ -160,3 +160,11 @@ def _register_kizezen():
 
 
 _register_kizezen()
+
+
+def _register_zabunex():
+    from .zabunex import ZabunexConfig, zabunex_plan
+    register_architecture("Zabunex", ZabunexConfig.from_dict, zabunex_plan)
+
+
+_register_zabunex()

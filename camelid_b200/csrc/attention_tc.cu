@@ -47,6 +47,9 @@ struct AtParams {
     float softcap;          // c > 0: the scaled score becomes c tanh(score / c) before mask and penalty
     int out_f32;            // the output rows are float (for a combination of maps that follows), else bfloat16
     int keep_first;         // > 0 (with a window): the sequence's first keep_first keys stay visible beside the window
+    const float* rel;       // [n_heads, n_rel] or null: added to the raw score (before the scale) by distance; distances of
+    int n_rel;              // n_rel - 1 and more share the last number
+    float out_scale;        // what the output rows are multiplied by
 };
 
 __device__ __forceinline__ uint32_t at_smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -414,6 +417,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap mapK, const __grid_co
 #pragma unroll
                 for (int c = 0; c < AT_KEYS; ++c) s[c] -= b1 * __log2f(fmaf(b2, fmaxf(d0 - (float)c, 0.f), 1.0f));
             }
+            if (ap.rel != nullptr) {
+                // neighbouring lanes are neighbouring tokens (of a head): their addresses are neighbours too
+                const float* by_distance = ap.rel + (size_t)(valid ? head : 0) * ap.n_rel;
+                const int d0 = pos - key0, last = ap.n_rel - 1;
+                if (d0 - (AT_KEYS - 1) >= last) {              // the whole page is as far as the table tells apart
+                    const float far = __ldg(by_distance + last);
+#pragma unroll
+                    for (int c = 0; c < AT_KEYS; ++c) s[c] += far;
+                } else {
+#pragma unroll
+                    for (int c = 0; c < AT_KEYS; ++c) s[c] += __ldg(by_distance + min(max(d0 - c, 0), last));
+                }
+            }
             {   // eight independent chains of three-input maxima, not one chain of 64
                 float mx8[8];
 #pragma unroll
@@ -505,7 +521,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap mapK, const __grid_co
                     const float m_ref = (m == -CUDART_INF_F) ? 0.f : m;
                     l += at_exp2(fminf(fmaf(ap.sink[head], 1.4426950408889634f, -m_ref * sl2), 126.0f));
                 }
-                float inv = valid ? 1.0f / l : 0.f;
+                float inv = valid ? ap.out_scale / l : 0.f;
                 if (ap.gate != nullptr && valid) inv *= 1.0f / (1.0f + __expf(-ap.gate[row * ap.gate_ld + ap.gate_col + head]));
                 const size_t out_at = row * p.out_stride + (size_t)(head * ap.maps + map) * HDV;
                 bf16* dst = (bf16*)p.out + out_at;
@@ -602,6 +618,8 @@ static int at_launch(const CUtensorMap& mk, const CUtensorMap& mv, AtParams ap, 
 // scaled score becomes c tanh(score / c). out_f32: the output rows are float (strides in elements either way).
 // head_dim: channels of a query and key (of one map); value_dim: of a value; 64 or 128 each. keep_first n > 0 (with a
 // window, no blocks): the first n keys of a sequence are visible to every later query of it, whatever the window.
+// rel (float [n_heads, n_rel] or null): score(i, j) = (q . k + rel[head][min(i - j, n_rel - 1)]) scale (a bias by distance,
+// divided by the scale beforehand); out_scale multiplies the output rows.
 extern "C" int cml_attn_prefill_tc_maps(const void* q, int q_stride, void* out, int out_stride, const void* k_pages,
                                         const void* v_pages, long n_pages, const int* block_table, int max_blocks,
                                         const int* tile_seq, const int* tile_q0, int n_tiles, const int* seq_row0,
@@ -609,9 +627,10 @@ extern "C" int cml_attn_prefill_tc_maps(const void* q, int q_stride, void* out, 
                                         int head_dim, int value_dim, int rows_per_tile, int heads_per_cta, int head_chunks,
                                         int window, float scale, const float* r1, const float* r2, int chunk,
                                         const float* sink, const float* gate, long gate_ld, int gate_col, int maps,
-                                        float softcap, int out_f32, int keep_first, int* err, void* stream) {
+                                        float softcap, int out_f32, int keep_first, const float* rel, int n_rel, float out_scale,
+                                        int* err, void* stream) {
     if (n_tiles <= 0) return 0;
-    if (keep_first < 0) return CML_ERR_BAD_SIZE;
+    if (keep_first < 0 || (rel && n_rel < 1)) return CML_ERR_BAD_SIZE;
     if (maps < 1 || !(softcap >= 0.f) || (softcap > 0.f && !(scale > 0.f))) return CML_ERR_BAD_SIZE;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return CML_ERR_BAD_SIZE;
     if (rows_per_tile < 1 || heads_per_cta < 1 || rows_per_tile * heads_per_cta > AT_ROWS) return CML_ERR_BAD_SIZE;
@@ -637,6 +656,7 @@ extern "C" int cml_attn_prefill_tc_maps(const void* q, int q_stride, void* out, 
     ap.r2 = (r1 && r2) ? r2 : nullptr;
     ap.chunk = chunk > 0 ? chunk : 0; ap.sink = sink; ap.gate = gate; ap.gate_ld = gate_ld; ap.gate_col = gate_col;
     ap.maps = maps; ap.softcap = softcap; ap.out_f32 = out_f32 ? 1 : 0; ap.keep_first = keep_first;
+    ap.rel = rel; ap.n_rel = n_rel; ap.out_scale = out_scale;
     cudaStream_t s = (cudaStream_t)stream;
     if (maps > 1) {          // the maps' outputs are subtracted from one another: the probabilities in two parts
         if (head_dim == 64) return value_dim == 64 ? at_launch<64, 64, true>(mk, mv, ap, n_tiles, s) : at_launch<64, 128, true>(mk, mv, ap, n_tiles, s);
@@ -656,7 +676,7 @@ extern "C" int cml_attn_prefill_tc_ext(const void* q, int q_stride, void* out, i
     return cml_attn_prefill_tc_maps(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, max_blocks, tile_seq,
                                     tile_q0, n_tiles, seq_row0, seq_start, seq_new, n_heads, n_kv_heads, head_dim, head_dim,
                                     rows_per_tile, heads_per_cta, head_chunks, window, scale, r1, r2, chunk, sink, gate, gate_ld,
-                                    gate_col, 1, 0.f, 0, 0, err, stream);
+                                    gate_col, 1, 0.f, 0, 0, nullptr, 0, 1.0f, err, stream);
 }
 
 extern "C" int cml_attn_prefill_tc_penalty(const void* q, int q_stride, void* out, int out_stride, const void* k_pages,

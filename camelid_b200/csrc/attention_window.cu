@@ -14,7 +14,8 @@
 // q in the compute type and writes k and v into their pages. The second gives a block to
 // every (row, head): lanes take keys for the scores (all in float), then columns of the
 // values; the softmax runs online over rounds of 32 keys, from the oldest visible key to the
-// row's own, whether the row came with a prompt or alone. With `keep_first` > 0 the first keep_first keys of the
+// row's own, whether the row came with a prompt or alone. `rel` (float [heads, n_rel] or null): a learned number per head and
+// distance, added to the scaled score (distances of n_rel - 1 and more share the last one). With `keep_first` > 0 the first keep_first keys of the
 // sequence stay visible beside the window; they come first in the order of the rounds. `v_stride`: channels between two
 // value rows of a page (Dv; or the key rows' size where the values are the first Dv channels of the key rows themselves).
 #include "common.cuh"
@@ -107,7 +108,10 @@ extern "C" int cml_qk_norm_kv_write(const float* proj, long ld, const void* q_w,
 // (n_splits matrices split_stride apart, added here in split order); the row is staged in shared memory, its sums
 // of squares taken on the way in. `extra` more columns behind v (the logits of an output gate) are copied, summed,
 // to extra_out [rows, extra]. `bias` (float, q, k, v and the extra columns; or null) is added to the summed row before
-// the norms; `rot_amp` multiplies every sine and cosine. A warp works on one head at a time, a lane on four neighbouring channels (two, or
+// the norms; `rot_amp` multiplies every sine and cosine. What QkvExtra adds: a short causal convolution over the q, k and v
+// channels of the summed rows before the norms (its inputs of the tokens before the step lie in a state per sequence),
+// values that are the k columns as they stand before the norm, and a factor on the queries that grows with the
+// position. A warp works on one head at a time, a lane on four neighbouring channels (two, or
 // one, where the head size allows no more), so that a warp's stores are one contiguous run.
 template <typename T> __device__ __forceinline__ void store_run(T* o, const float* v, int n);
 template <> __device__ __forceinline__ void store_run<float>(float* o, const float* v, int n) {
@@ -126,15 +130,57 @@ template <> __device__ __forceinline__ void store_run<bf16>(bf16* o, const float
     }
 }
 
-template <typename T, typename TW, int THREADS>
-__global__ void __launch_bounds__(THREADS, THREADS <= 256 ? 5 : 1)
+struct QkvExtra {
+    const float* conv_w;        // [taps, q + k + v columns] (the last tap the current token's), or null
+    float* conv_state;          // [slots, max(taps - 1, 1), q + k + v columns]: the inputs of the tokens before the step
+    int taps;
+    int update_state;           // every sequence of the step brings one row: the state moves on by it here
+    const int* seq_row0;
+    const int* seq_slot;
+    int share_v;                // the values are the k columns before the norm (no v columns; Dv == D)
+    float temp_coef;            // q times 1 + temp_coef ln(floor((position + 1) / temp_every) + 1); 0: as it is
+    float temp_every;
+};
+
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void fma4(float4& a, const float4& w, const float4& u) {
+    a.x = fmaf(w.x, u.x, a.x); a.y = fmaf(w.y, u.y, a.y); a.z = fmaf(w.z, u.z, a.z); a.w = fmaf(w.w, u.w, a.w);
+}
+// the sum over the splits, eight at a time: unconditional loads (of a valid place), all in flight before the first add; the
+// adds stay in split order
+__device__ __forceinline__ float4 split_sum4(const float* p, int n_splits, long stride) {
+    float4 v = ld4(p);
+    for (int s0 = 1; s0 < n_splits; s0 += 8) {
+        float4 t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = ld4(p + (size_t)min(s0 + k, n_splits - 1) * stride);
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            if (s0 + k < n_splits) { v.x += t[k].x; v.y += t[k].y; v.z += t[k].z; v.w += t[k].w; }
+    }
+    return v;
+}
+__device__ __forceinline__ float split_sum1(const float* p, int n_splits, long stride) {
+    float v = p[0];
+    for (int s0 = 1; s0 < n_splits; s0 += 8) {
+        float t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = p[(size_t)min(s0 + k, n_splits - 1) * stride];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += s0 + k < n_splits ? t[k] : 0.f;
+    }
+    return v;
+}
+
+template <typename T, typename TW, int THREADS, bool CONV>
+__global__ void __launch_bounds__(THREADS, THREADS > 256 ? 1 : CONV ? 3 : 5)
 qkv_prepare_kernel(const float* __restrict__ proj, long ld, int n_splits, long split_stride, int extra,
                    float* __restrict__ extra_out, const TW* __restrict__ q_w, const TW* __restrict__ k_w, int norm_mode, float eps,
                    const float* __restrict__ inv_freq, int rot_dim, int pairing, const int* __restrict__ row_seq,
                    const int* __restrict__ row_pos, const int* __restrict__ table, int max_blocks, T* __restrict__ q_out,
                    T* __restrict__ k_pages, T* __restrict__ v_pages, int heads, int kv_heads, int D, int Dv,
-                   const float* __restrict__ bias, float rot_amp) {
-    __shared__ float red[2][32];
+                   const float* __restrict__ bias, float rot_amp, const QkvExtra ex) {
+    __shared__ float red[2][32], temp;
     __shared__ float2 turn[128];                                // (cosine, sine) of the row's angles, shared by all heads
     extern __shared__ __align__(16) float x[];                 // the row: q, k, v, the extra columns
     pdl_wait();
@@ -143,22 +189,43 @@ qkv_prepare_kernel(const float* __restrict__ proj, long ld, int n_splits, long s
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     constexpr int NWARPS = THREADS / 32;
     const int qw = heads * D, kw = kv_heads * D, vw = kv_heads * Dv;
-    const int total = qw + kw + vw + extra;
+    const int conv_cols = qw + kw + (ex.share_v ? 0 : vw);
+    const int total = conv_cols + extra;
     const float* src = proj + (size_t)r * ld;
+    const int pos = row_pos[r], seq = row_seq[r];
+    const int taps = CONV ? ex.taps : 0;
+    const int inside = CONV ? r - ex.seq_row0[seq] : 0;         // rows of this step before this one, of the same sequence
+    float* st = CONV ? ex.conv_state + (size_t)ex.seq_slot[seq] * max(taps - 1, 1) * conv_cols : nullptr;
     float sq = 0.f, sk = 0.f;                                   // sums of squares of the q and the k columns
-    if (((ld | split_stride | (long)total) & 3) == 0 && (((uintptr_t)proj) & 15) == 0) {
+    if (((ld | split_stride | (long)total | (long)conv_cols) & 3) == 0 && (((uintptr_t)proj) & 15) == 0) {
         for (int c = threadIdx.x * 4; c < total; c += THREADS * 4) {
-            float4 v = *reinterpret_cast<const float4*>(src + c);
-            // the other splits eight at a time: unconditional loads (of a valid place), all in flight before the first
-            // add; the adds stay in split order
-            for (int s0 = 1; s0 < n_splits; s0 += 8) {
-                float4 t[8];
+            float4 v = split_sum4(src + c, n_splits, split_stride);
+            if (CONV && c < conv_cols) {
+                float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+                fma4(acc, ld4(ex.conv_w + (size_t)(taps - 1) * conv_cols + c), v);
+                for (int b0 = 1; b0 < taps; b0 += 3) {          // three tokens back at a time, their loads in flight together
+                    float4 u[3], w[3];
 #pragma unroll
-                for (int k = 0; k < 8; ++k)
-                    t[k] = *reinterpret_cast<const float4*>(src + (size_t)min(s0 + k, n_splits - 1) * split_stride + c);
+                    for (int k = 0; k < 3; ++k) {
+                        const int back = b0 + k;
+                        const bool ok = back < taps && back <= pos, here = back <= inside;
+                        u[k] = ld4(!ok ? src + c : here ? src - (size_t)back * ld + c : st + (size_t)(taps - 1 + inside - back) * conv_cols + c);
+                        w[k] = ld4(ex.conv_w + (size_t)max(taps - 1 - back, 0) * conv_cols + c);
+                        if (ok && here && n_splits > 1) u[k] = split_sum4(src - (size_t)back * ld + c, n_splits, split_stride);
+                        if (!ok) w[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    }
 #pragma unroll
-                for (int k = 0; k < 8; ++k)
-                    if (s0 + k < n_splits) { v.x += t[k].x; v.y += t[k].y; v.z += t[k].z; v.w += t[k].w; }
+                    for (int k = 0; k < 3; ++k) fma4(acc, w[k], u[k]);
+                }
+                if (ex.update_state && taps > 1) {              // drop the oldest input, keep this row's
+                    for (int j = 0; j + 2 < taps; ++j) {
+                        float4 t = ld4(st + (size_t)(j + 1) * conv_cols + c);
+                        if (pos + j + 2 < taps) t = make_float4(0.f, 0.f, 0.f, 0.f);
+                        *reinterpret_cast<float4*>(st + (size_t)j * conv_cols + c) = t;
+                    }
+                    *reinterpret_cast<float4*>(st + (size_t)(taps - 2) * conv_cols + c) = v;
+                }
+                v = acc;
             }
             if (bias != nullptr) {                              // the projections' biases, after the sums
                 const float4 b = *reinterpret_cast<const float4*>(bias + c);
@@ -174,13 +241,20 @@ qkv_prepare_kernel(const float* __restrict__ proj, long ld, int n_splits, long s
         }
     } else {
         for (int c = threadIdx.x; c < total; c += THREADS) {
-            float v = src[c];
-            for (int s0 = 1; s0 < n_splits; s0 += 8) {
-                float t[8];
-#pragma unroll
-                for (int k = 0; k < 8; ++k) t[k] = src[(size_t)min(s0 + k, n_splits - 1) * split_stride + c];
-#pragma unroll
-                for (int k = 0; k < 8; ++k) v += s0 + k < n_splits ? t[k] : 0.f;
+            float v = split_sum1(src + c, n_splits, split_stride);
+            if (CONV && c < conv_cols) {
+                float acc = ex.conv_w[(size_t)(taps - 1) * conv_cols + c] * v;
+                for (int back = 1; back < taps && back <= pos; ++back) {
+                    const float u = back <= inside ? split_sum1(src - (size_t)back * ld + c, n_splits, split_stride)
+                                                   : st[(size_t)(taps - 1 + inside - back) * conv_cols + c];
+                    acc = fmaf(ex.conv_w[(size_t)(taps - 1 - back) * conv_cols + c], u, acc);
+                }
+                if (ex.update_state && taps > 1) {
+                    for (int j = 0; j + 2 < taps; ++j)
+                        st[(size_t)j * conv_cols + c] = pos + j + 2 >= taps ? st[(size_t)(j + 1) * conv_cols + c] : 0.f;
+                    st[(size_t)(taps - 2) * conv_cols + c] = v;
+                }
+                v = acc;
             }
             if (bias != nullptr) v += bias[c];
             x[c] = v;
@@ -188,13 +262,14 @@ qkv_prepare_kernel(const float* __restrict__ proj, long ld, int n_splits, long s
             else if (c < qw + kw) sk = fmaf(v, v, sk);
         }
     }
-    const int pos = row_pos[r];
-    const int page = table[(size_t)row_seq[r] * max_blocks + pos / CML_PAGE];
+    const int page = table[(size_t)seq * max_blocks + pos / CML_PAGE];
     for (int i = threadIdx.x; i < rot_dim / 2; i += THREADS) {
         float sn, cs;
         sincosf((float)pos * inv_freq[i], &sn, &cs);
         turn[i] = make_float2(cs * rot_amp, sn * rot_amp);
     }
+    if (threadIdx.x == 0 && ex.temp_coef != 0.f)                // what the queries are multiplied by
+        temp = 1.0f + ex.temp_coef * logf((float)floor((double)(pos + 1) / (double)ex.temp_every) + 1.0f);
     if (norm_mode == 2) {                                       // both sums over the block with one barrier
         sq = warp_sum(sq);
         sk = warp_sum(sk);
@@ -254,13 +329,18 @@ qkv_prepare_kernel(const float* __restrict__ proj, long ld, int n_splits, long s
                     }
                 }
             }
+            if (is_q && ex.temp_coef != 0.f) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) out[i] *= temp;
+            }
             store_run<T>(o + d, out, run);
         }
     }
     if (page >= 0) {
         T* v_row = v_pages + ((size_t)page * kv_heads * CML_PAGE + pos % CML_PAGE) * Dv;
-        const float* xv = x + qw + kw;
-        if ((Dv & 3) == 0 && ((qw + kw) & 3) == 0) {
+        const int v_at = ex.share_v ? qw : qw + kw;
+        const float* xv = x + v_at;
+        if ((Dv & 3) == 0 && (v_at & 3) == 0) {
             for (int c = threadIdx.x * 4; c < vw; c += THREADS * 4) {
                 const int g = c / Dv, e = c - g * Dv;
                 const float4 v = *reinterpret_cast<const float4*>(xv + c);
@@ -280,8 +360,14 @@ extern "C" int cml_qkv_prepare(const float* proj, long ld, int n_splits, long sp
                                const void* q_w, const void* k_w, int w_dtype, int norm_mode, float eps, const float* inv_freq,
                                int rot_dim, int pairing, const int* row_seq, const int* row_pos, const int* table,
                                int max_blocks, void* q_out, void* k_pages, void* v_pages, int dtype, int rows, int heads,
-                               int kv_heads, int D, int Dv, const float* bias, float rot_amp, void* stream) {
+                               int kv_heads, int D, int Dv, const float* bias, float rot_amp, const float* conv_w,
+                               float* conv_state, int taps, int update_state, const int* seq_row0, const int* seq_slot,
+                               int share_v, float temp_coef, float temp_every, void* stream) {
     if (rows <= 0) return 0;
+    if (conv_w && (taps < 1 || bias || !conv_state || !seq_row0 || !seq_slot)) return CML_ERR_BAD_SIZE;
+    if ((share_v && D != Dv) || (temp_coef != 0.f && !(temp_every > 0.f))) return CML_ERR_BAD_SIZE;
+    if ((((uintptr_t)conv_w) | ((uintptr_t)conv_state)) & 15) return CML_ERR_BAD_ALIGN;
+    const QkvExtra ex = {conv_w, conv_state, taps, update_state, seq_row0, seq_slot, share_v, temp_coef, temp_every};
     if (rot_dim < 0 || rot_dim > D || rot_dim > 256 || (rot_dim & 1) || norm_mode < 0 || norm_mode > 2) return CML_ERR_BAD_SIZE;
     if (n_splits < 1 || extra < 0) return CML_ERR_BAD_SIZE;
     // the vector stores want aligned rows: the outputs' bases come 16-byte aligned from the allocator, the sizes decide the rest
@@ -290,17 +376,18 @@ extern "C" int cml_qkv_prepare(const float* proj, long ld, int n_splits, long sp
     const size_t smem = (size_t)(heads * D + kv_heads * (D + Dv) + extra + 4) * sizeof(float);
     if (smem > 200 * 1024) return CML_ERR_BAD_SIZE;
     const bool few = rows <= 128;                               // one-token steps: more threads per row
-#define QP_LAUNCH(T_, TW_, N_)                                                                                             \
+#define QP_LAUNCH(T_, TW_, N_, C_)                                                                                             \
     {                                                                                                                      \
-        if (smem > 48 * 1024 && cml_allow_smem<qkv_prepare_kernel<T_, TW_, N_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE; \
-        launch_pdl(qkv_prepare_kernel<T_, TW_, N_>, dim3(rows), dim3(N_), smem, s, proj, ld, n_splits, split_stride, extra, \
+        if (smem > 48 * 1024 && cml_allow_smem<qkv_prepare_kernel<T_, TW_, N_, C_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE; \
+        launch_pdl(qkv_prepare_kernel<T_, TW_, N_, C_>, dim3(rows), dim3(N_), smem, s, proj, ld, n_splits, split_stride, extra, \
                    extra_out, (const TW_*)q_w, (const TW_*)k_w, norm_mode, eps, inv_freq, rot_dim, pairing, row_seq, row_pos, \
-                   table, max_blocks, (T_*)q_out, (T_*)k_pages, (T_*)v_pages, heads, kv_heads, D, Dv, bias, rot_amp);       \
+                   table, max_blocks, (T_*)q_out, (T_*)k_pages, (T_*)v_pages, heads, kv_heads, D, Dv, bias, rot_amp, ex);   \
         return cml_launch_status();                                                                                        \
     }
 #define QP_CASE(T_, TW_, D_, DW_)                                                                                          \
     if (dtype == D_ && w_dtype == DW_) {                                                                                   \
-        if (few) QP_LAUNCH(T_, TW_, 1024) else QP_LAUNCH(T_, TW_, 256)                                                     \
+        if (conv_w) { if (few) QP_LAUNCH(T_, TW_, 512, true) else QP_LAUNCH(T_, TW_, 256, true) }                          \
+        if (few) QP_LAUNCH(T_, TW_, 1024, false) else QP_LAUNCH(T_, TW_, 256, false)                                       \
     }
     QP_CASE(float, float, CML_DTYPE_F32, CML_DTYPE_F32)
     QP_CASE(bf16, bf16, CML_DTYPE_BF16, CML_DTYPE_BF16)
@@ -354,7 +441,10 @@ struct AwExtra {
     float softcap;          // 0: none
     float lambda;           // MAPS == 2: the factor of the second map
     float norm_eps;         // MAPS == 2: eps of the norm of the difference
-    float out_scale;        // MAPS == 2: what the normed difference is multiplied by
+    float out_scale;        // what the head's output (MAPS == 2: the normed difference) is multiplied by
+    const float* rel;       // [heads, n_rel] or null: added to the scaled score by distance
+    int n_rel;
+    long ldo;               // elements between two output rows
 };
 
 template <typename T, int NV, int MAPS>    // NV: value columns per lane, Dv <= 32 * NV
@@ -458,6 +548,7 @@ __global__ void __launch_bounds__(512, 1) window_attention_kernel(const T* __res
                     float v = dot * scale;
                     if (ex.softcap > 0.f) v = ex.softcap * tanhf(v / ex.softcap);
                     if (r1) v -= p1 * log1pf(p2 * (float)(i - j));
+                    if (ex.rel) v += ex.rel[(size_t)hd * ex.n_rel + min(i - j, ex.n_rel - 1)];
                     sc[mp] = v;
                 }
             }
@@ -535,7 +626,7 @@ __global__ void __launch_bounds__(512, 1) window_attention_kernel(const T* __res
         top[mp] = tp;
         inv[mp] = 1.0f / total;
     }
-    T* o = out + ((size_t)r * heads + hd) * Dv;
+    T* o = out + (size_t)r * ex.ldo + (size_t)hd * Dv;
     const float* gt = gate ? gate + (size_t)r * ldg + gate_col + (gate_per_head ? hd : hd * Dv) : nullptr;
     const int gstep = gate_per_head ? 0 : 1;
     auto merged = [&](int mp, int c) -> float {
@@ -548,7 +639,7 @@ __global__ void __launch_bounds__(512, 1) window_attention_kernel(const T* __res
     };
     if (MAPS == 1) {
         for (int c = threadIdx.x; c < Dv; c += blockDim.x)
-            o[c] = from_f32<T>(merged(0, c) * (gt ? sigmoid_w(gt[c * gstep]) : 1.0f));
+            o[c] = from_f32<T>(merged(0, c) * ex.out_scale * (gt ? sigmoid_w(gt[c * gstep]) : 1.0f));
         return;
     }
     // the difference of the two maps, normed over the head's channels: the differences stand behind the warps' parts
@@ -570,8 +661,9 @@ extern "C" int cml_window_attention(const void* q, const void* k_pages, const vo
                                     const float* gate, long ldg, int gate_col, void* out, int rows, int heads, int kv_heads,
                                     int D, int Dv, int window, float scale, int chunk, const float* sink, int gate_per_head,
                                     int maps, float softcap, float lambda, float norm_eps, float out_scale, int keep_first,
-                                    int v_stride, void* stream) {
+                                    int v_stride, const float* rel, int n_rel, long ldo, void* stream) {
     if (rows <= 0) return 0;
+    if ((rel && n_rel < 1) || ldo < (long)heads * Dv) return CML_ERR_BAD_SIZE;
     if (Dv > 32 * AW_MAX_VREGS || D < 1 || heads % kv_heads || (maps != 1 && maps != 2)) return CML_ERR_BAD_SIZE;
     if (keep_first < 0 || v_stride < Dv || (maps == 2 && Dv > 256)) return CML_ERR_BAD_SIZE;
     // warps per (row, head): one per round of 32 keys of the window, at most 16 (8 without a window); fixed by
@@ -585,7 +677,7 @@ extern "C" int cml_window_attention(const void* q, const void* k_pages, const vo
     const size_t smem = (size_t)(((maps * D + 3) & ~3) + nw * maps * (Dv + 2) + (maps > 1 ? ((Dv + 3) & ~3) + 32 : 0)) * sizeof(float);
     if (smem > 48 * 1024 || (long)rows * heads > 0x7fffffffL) return CML_ERR_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
-    const AwExtra ex = {softcap, lambda, norm_eps, out_scale};
+    const AwExtra ex = {softcap, lambda, norm_eps, out_scale, rel, n_rel, ldo};
 #define AW_CASE(T_, NV_, MP_)                                                                                               \
     launch_pdl(window_attention_kernel<T_, NV_, MP_>, grid, dim3(32 * nw), smem, s, (const T_*)q, (const T_*)k_pages, (const T_*)v_pages, \
                table, max_blocks, row_seq, row_pos, r1, r2, gate, ldg, gate_col, (T_*)out, heads, kv_heads, D, Dv, window, scale, \

@@ -64,7 +64,7 @@ _SIGNATURES = {
                                                    c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                    c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
                                                    c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_float, c_int, c_int,
-                                                   c_void_p, c_void_p],
+                                                   c_void_p, c_int, c_float, c_void_p, c_void_p],
     ("attention_window", "cml_maps_difference"): [c_void_p, c_long, c_void_p, c_long, c_int, c_long, c_int, c_int, c_float, c_float,
                                                   c_float, c_void_p],
     ("attention_tc", "cml_attn_prefill_tc_penalty"): [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_void_p,
@@ -141,10 +141,11 @@ _SIGNATURES = {
     ("attention_window", "cml_window_attention"): [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                                    c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p, c_int, c_int, c_int,
                                                    c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_int, c_float, c_float,
-                                                   c_float, c_float, c_int, c_int, c_void_p],
+                                                   c_float, c_float, c_int, c_int, c_void_p, c_int, c_long, c_void_p],
     ("attention_window", "cml_qkv_prepare"): [c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int,
                                               c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                              c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
+                                              c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
+                                              c_void_p, c_void_p, c_int, c_float, c_float, c_void_p],
     ("attention_latent", "cml_latent_prepare"): [c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p,
                                                  c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
@@ -156,6 +157,13 @@ _SIGNATURES = {
                                                 c_int, c_float, c_void_p, c_int, c_int, c_long, c_int, c_void_p],
     ("recurrence", "cml_retention_scan"): [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    ("recurrence", "cml_ssm_inputs"): [c_void_p, c_long, c_int, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                                       c_int, c_int, c_void_p],
+    ("recurrence", "cml_ssm_scan"): [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p,
+                                     c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    ("recurrence", "cml_gated_group_norm"): [c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int,
+                                             c_float, c_void_p],
     ("recurrence", "cml_rotate_rows"): [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
                                         c_int, c_float, c_void_p],
     ("token_ops", "cml_tanh_columns"): [c_void_p, c_long, c_int, c_long, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -842,6 +850,59 @@ def delta_chunk_scan(chunks: torch.Tensor, state: torch.Tensor, seq_row0, seq_ne
                                                      _p(out), n_seqs, heads, key_dim, value_dim, _stream()), "delta_chunk_scan")
 
 
+def ssm_inputs(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+               state: torch.Tensor, row_seq, row_pos, seq_row0, seq_slot, out: torch.Tensor, gates: torch.Tensor, inner: int,
+               z_out=None, update_state: bool = False):
+    """What the state-space recurrence reads, from ``proj`` (float32 [rows, n] or split sums [splits, rows, n], added here): columns
+    z (``inner``), the convolved channels (x, B, C), one step-size input per head. ``conv_w`` float32 [taps, channels], ``conv_b``
+    [channels]; ``state`` float32 [slots, max(taps - 1, 1), channels]: the inputs of the tokens before the step (moved on here
+    with ``update_state``, where every sequence brings one row). ``out`` float32 [rows, channels] = silu(conv + bias); ``gates``
+    float32 [rows, 2 heads] = dt = softplus(in + dt_bias), then exp(-exp(a_log) dt); ``z_out`` float32 [rows, inner] or None."""
+    _dev(proj, conv_w, conv_b, dt_bias, a_log, state, row_seq, row_pos, seq_row0, seq_slot, out, gates, z_out)
+    if proj.dim() == 2:
+        proj = proj.unsqueeze(0)
+    taps, channels = conv_w.shape
+    heads, rows = dt_bias.numel(), out.shape[0]
+    for t in (proj, conv_w, conv_b, dt_bias, a_log, state, out, gates):
+        assert t.dtype == torch.float32 and t.stride(-1) == 1
+    assert proj.shape[1] == rows and proj.shape[2] >= inner + channels + heads and a_log.numel() == heads and conv_b.numel() == channels
+    assert conv_w.is_contiguous() and state.is_contiguous() and state.shape[1:] == (max(taps - 1, 1), channels)
+    assert out.is_contiguous() and out.shape[1] == channels and gates.is_contiguous() and gates.shape == (rows, 2 * heads)
+    assert z_out is None or (z_out.dtype == torch.float32 and z_out.is_contiguous() and z_out.shape == (rows, inner))
+    _check(_fn("recurrence", "cml_ssm_inputs")(_p(proj), proj.stride(1), proj.shape[0], proj.stride(0), _p(conv_w), _p(conv_b), _p(dt_bias),
+                                               _p(a_log), _p(state), 1 if update_state else 0, _p(row_seq), _p(row_pos), _p(seq_row0),
+                                               _p(seq_slot), _p(out), _p(gates), _p(z_out), rows, inner, channels, heads, taps,
+                                               _stream()), "ssm_inputs")
+
+
+def ssm_scan(rows_in: torch.Tensor, cols: tuple, gates: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor, seq_row0, seq_new,
+             seq_start, seq_slot, out: torch.Tensor, n_seqs: int, heads: int, groups: int, key_dim: int, value_dim: int):
+    """The state-space recurrence over each sequence's new rows: S <- decay S + dt B x^T, out = S^T C + D x per head. ``cols``:
+    columns of x (``heads`` x ``value_dim``), B and C (``groups`` x ``key_dim``, each shared by heads / groups heads) in ``rows_in``;
+    ``gates`` [rows, 2 heads]: dt, then the decays; ``d_skip`` [heads]; ``state`` float32 [slots, heads, value_dim, key_dim]
+    (column by column) is read and replaced; ``out`` float32 [rows, heads * value_dim]."""
+    _dev(rows_in, gates, d_skip, state, seq_row0, seq_new, seq_start, seq_slot, out)
+    for t in (rows_in, gates, d_skip, state, out):
+        assert t.dtype == torch.float32 and t.stride(-1) == 1
+    assert d_skip.numel() == heads and gates.shape[1] == 2 * heads
+    assert state.is_contiguous() and state.shape[1:] == (heads, value_dim, key_dim) and out.is_contiguous() and out.shape[1] == heads * value_dim
+    x_col, b_col, c_col = cols
+    _check(_fn("recurrence", "cml_ssm_scan")(_p(rows_in), rows_in.stride(0), x_col, b_col, c_col, _p(gates), gates.stride(0), _p(d_skip),
+                                             _p(state), _p(seq_row0), _p(seq_new), _p(seq_start), _p(seq_slot), _p(out), n_seqs, heads,
+                                             groups, key_dim, value_dim, _stream()), "ssm_scan")
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, groups: int, eps: float, out: torch.Tensor):
+    """v = y * silu(z), each of ``groups`` equal parts of a row divided by its root mean square, times ``w`` (float32 [width]), to
+    ``out`` in the compute type (rows of any stride). y float32 [rows, width] contiguous, z float32 rows of any stride."""
+    _dev(y, z, w, out)
+    rows, width = y.shape
+    assert y.dtype == z.dtype == w.dtype == torch.float32 and y.is_contiguous() and z.stride(1) == 1 and z.shape == (rows, width)
+    assert w.numel() == width and w.is_contiguous() and width % groups == 0 and out.shape == (rows, width) and out.stride(1) == 1
+    _check(_fn("recurrence", "cml_gated_group_norm")(_p(y), _p(z), z.stride(0), _p(w), _p(out), out.stride(0), dtype_code(out.dtype), rows,
+                                                     width, groups, float(eps), _stream()), "gated_group_norm")
+
+
 def rotate_rows_(x: torch.Tensor, col0: int, heads: int, head_dim: int, rotary_dim: int, interleaved: bool, inv_freq, amp: float,
                  row_pos, scaled_from: int | None = None, scale: float = 1.0):
     """In place on float32 rows: the ``heads`` heads of ``head_dim`` channels from column ``col0`` have their first
@@ -900,8 +961,10 @@ def qk_norm_kv_write(proj: torch.Tensor, q_w, k_w, eps: float, row_seq, row_pos,
 def window_attention(q, k_pages, v_pages, table, row_seq, row_pos, r1, r2, gate, gate_col: int, out, heads: int,
                      kv_heads: int, key_dim: int, value_dim: int, window: int, scale: float, chunk: int = 0, sink=None,
                      gate_per_head: bool = False, softcap: float = 0.0, difference=None, keep_first: int = 0,
-                     values_in_keys: bool = False):
-    """``softcap`` c > 0: the scaled score becomes c tanh(score / c). ``difference`` = (lambda, eps, out_scale): every head
+                     values_in_keys: bool = False, distance_bias=None, out_scale: float = 1.0):
+    """``distance_bias`` (float32 [heads, n]): added to the scaled score of the key at distance i - j (distances of n - 1 and
+    more share the last number). ``out_scale`` multiplies the heads. ``out``: rows of any stride.
+    ``softcap`` c > 0: the scaled score becomes c tanh(score / c). ``difference`` = (lambda, eps, out_scale): every head
     has two score maps (q and the key rows hold both, ``key_dim`` channels each), out = rmsnorm_eps(a1 - lambda a2) * out_scale
     per head (differential attention).
     out[r, head] = softmax_j((q . k_j) scale - r1 ln(1 + r2 (i - j))) V over the last ``window`` keys
@@ -913,7 +976,10 @@ def window_attention(q, k_pages, v_pages, table, row_seq, row_pos, r1, r2, gate,
     _dev(q, k_pages, v_pages, table, row_seq, row_pos, r1, r2, gate, out, sink)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == heads and sink.is_contiguous())
     rows = q.shape[0]
-    assert q.is_contiguous() and out.is_contiguous() and q.dtype == out.dtype == k_pages.dtype == v_pages.dtype
+    assert q.is_contiguous() and out.stride(1) == 1 and q.dtype == out.dtype == k_pages.dtype == v_pages.dtype
+    if distance_bias is not None:
+        _dev(distance_bias)
+        assert distance_bias.dtype == torch.float32 and distance_bias.is_contiguous() and distance_bias.shape[0] == heads
     maps = 2 if difference is not None else 1
     lam, d_eps, d_scale = difference if difference is not None else (0.0, 0.0, 1.0)
     assert out.shape == (rows, heads * value_dim) and q.shape[1] == maps * heads * key_dim
@@ -930,14 +996,19 @@ def window_attention(q, k_pages, v_pages, table, row_seq, row_pos, r1, r2, gate,
         _p(q), _p(k_pages), _p(v_pages), dtype_code(q.dtype), _p(table), table.shape[1], _p(row_seq), _p(row_pos), _p(r1),
         _p(r2), _p(gate), gate.stride(0) if gate is not None else 0, gate_col, _p(out), rows, heads, kv_heads, key_dim,
         value_dim, int(window or 0), float(scale), int(chunk or 0), _p(sink), 1 if gate_per_head else 0, maps, float(softcap or 0.0),
-        float(lam), float(d_eps), float(d_scale), int(keep_first or 0), maps * key_dim if values_in_keys else value_dim,
-        _stream()), "window_attention")
+        float(lam), float(d_eps), float(d_scale) * float(out_scale), int(keep_first or 0), maps * key_dim if values_in_keys else value_dim,
+        _p(distance_bias), distance_bias.shape[1] if distance_bias is not None else 0, out.stride(0), _stream()), "window_attention")
 
 
 def qkv_prepare(proj: torch.Tensor, q_w, k_w, norm_mode: int, eps: float, inv_freq, rotary_dim: int, interleaved: bool,
                 row_seq, row_pos, table, q_out, k_pages, v_pages, heads: int, kv_heads: int, key_dim: int, value_dim: int,
-                extra_out=None, bias=None, amplitude: float = 1.0):
-    """``bias`` (float32, one number per column of q, k, v and the extra columns): added to the summed row before the norms;
+                extra_out=None, bias=None, amplitude: float = 1.0, conv=None, share_values: bool = False, temperature=None):
+    """``conv`` = (weights float32 [taps, q + k + v columns], state float32 [slots, max(taps - 1, 1), the same columns], seq_row0,
+    seq_slot, update_state): a short causal convolution over the summed q, k and v columns before the norms; the state holds
+    the inputs of the tokens before the step and moves on here with ``update_state`` (where every sequence brings one row).
+    ``share_values``: the values are the k columns as they stand before the norm; ``proj`` has no v columns. ``temperature`` =
+    (coef, every): q times 1 + coef ln(floor((position + 1) / every) + 1).
+    ``bias`` (float32, one number per column of q, k, v and the extra columns): added to the summed row before the norms;
     ``amplitude`` multiplies every sine and cosine.
     From ``proj`` (float32 rows: q, k, v; [rows, n] or split sums [splits, rows, n], added here): RMS norm of q and k (``norm_mode`` 0 none, 1 per head with weights
     [key_dim], 2 over the whole projection with weights [heads * key_dim] and [kv_heads * key_dim]), then the
@@ -951,7 +1022,9 @@ def qkv_prepare(proj: torch.Tensor, q_w, k_w, norm_mode: int, eps: float, inv_fr
     assert proj.dtype == torch.float32 and proj.stride(2) == 1 and proj.shape[1] == rows
     extra = extra_out.shape[1] if extra_out is not None else 0
     assert extra_out is None or (extra_out.dtype == torch.float32 and extra_out.is_contiguous() and extra_out.shape[0] == rows)
-    assert proj.shape[2] >= heads * key_dim + kv_heads * (key_dim + value_dim) + extra
+    v_cols = 0 if share_values else kv_heads * value_dim
+    assert proj.shape[2] >= heads * key_dim + kv_heads * key_dim + v_cols + extra
+    assert not share_values or key_dim == value_dim
     assert q_out.is_contiguous() and q_out.shape[1] == heads * key_dim and k_pages.dtype == q_out.dtype == v_pages.dtype
     assert k_pages.is_contiguous() and v_pages.is_contiguous()
     assert k_pages.shape[1:] == (kv_heads, PAGE, key_dim) and v_pages.shape[1:] == (kv_heads, PAGE, value_dim)
@@ -963,12 +1036,23 @@ def qkv_prepare(proj: torch.Tensor, q_w, k_w, norm_mode: int, eps: float, inv_fr
     if bias is not None:
         _dev(bias)
         assert bias.dtype == torch.float32 and bias.is_contiguous()
-        assert bias.numel() == heads * key_dim + kv_heads * (key_dim + value_dim) + extra
+        assert bias.numel() == heads * key_dim + kv_heads * key_dim + v_cols + extra
+    conv_w = conv_state = conv_row0 = conv_slot = None
+    taps = update = 0
+    if conv is not None:
+        conv_w, conv_state, conv_row0, conv_slot, update = conv
+        _dev(conv_w, conv_state, conv_row0, conv_slot)
+        taps, cols = conv_w.shape
+        assert bias is None and cols == heads * key_dim + kv_heads * key_dim + v_cols
+        assert conv_w.dtype == conv_state.dtype == torch.float32 and conv_w.is_contiguous() and conv_state.is_contiguous()
+        assert conv_state.shape[1:] == (max(taps - 1, 1), cols)
+    coef, every = temperature if temperature is not None else (0.0, 1.0)
     _check(_fn("attention_window", "cml_qkv_prepare")(
         _p(proj), proj.stride(1), proj.shape[0], proj.stride(0), extra, _p(extra_out), _p(q_w), _p(k_w), dtype_code(q_w.dtype) if norm_mode else dtype_code(q_out.dtype), int(norm_mode),
         float(eps), _p(inv_freq), int(rotary_dim), 1 if interleaved else 0, _p(row_seq), _p(row_pos), _p(table), table.shape[1],
         _p(q_out), _p(k_pages), _p(v_pages), dtype_code(q_out.dtype), rows, heads, kv_heads, key_dim, value_dim, _p(bias),
-        float(amplitude), _stream()), "qkv_prepare")
+        float(amplitude), _p(conv_w), _p(conv_state), taps, 1 if update else 0, _p(conv_row0), _p(conv_slot), 1 if share_values else 0,
+        float(coef), float(every), _stream()), "qkv_prepare")
 
 
 def latent_prepare(proj: torch.Tensor, c_w, eps: float, inv_freq, interleaved: bool, amplitude: float, row_seq,
@@ -1460,8 +1544,10 @@ def attn_tc_usable(q: torch.Tensor, out: torch.Tensor, head_dim: int, value_dim:
 def attn_prefill_tc(q, out, k_pages, v_pages, block_table, tile_seq, tile_q0, n_tiles, seq_row0, seq_start, seq_new,
                     n_heads, n_kv_heads, head_dim, rows_per_tile, heads_per_cta, head_chunks, window, scale, err,
                     r1=None, r2=None, chunk: int = 0, sink=None, head_gate=None, gate_col: int = 0, maps: int = 1,
-                    softcap: float = 0.0, value_dim: int | None = None, keep_first: int = 0):
-    """``keep_first`` n (with ``window``): the first n keys of a sequence stay visible to all its later queries.
+                    softcap: float = 0.0, value_dim: int | None = None, keep_first: int = 0, raw_bias=None, out_scale: float = 1.0):
+    """``raw_bias`` (float32 [heads, n]): score = (q . k + raw_bias[head][min(i - j, n - 1)]) scale (a bias by distance, divided
+    by the scale). ``out_scale`` multiplies the output rows.
+    ``keep_first`` n (with ``window``): the first n keys of a sequence stay visible to all its later queries.
     bfloat16 prefill attention of packed query rows over the paged cache with tcgen05.mma. ``r1``, ``r2``
     (float32 [heads]): the score of key j for query i loses r1 ln(1 + r2 (i - j)). ``chunk``: queries see only the
     keys of their own block of ``chunk`` positions. ``sink`` (float32 [heads]): one more term exp(sink) in the
@@ -1484,13 +1570,16 @@ def attn_prefill_tc(q, out, k_pages, v_pages, block_table, tile_seq, tile_q0, n_
     assert v_pages.shape == (k_pages.shape[0], n_kv_heads, PAGE, value_dim)
     if r1 is not None:
         assert r1.dtype == torch.float32 and r2.dtype == torch.float32 and r1.numel() == n_heads and r2.numel() == n_heads
+    if raw_bias is not None:
+        _dev(raw_bias)
+        assert raw_bias.dtype == torch.float32 and raw_bias.is_contiguous() and raw_bias.shape[0] == n_heads
     _check(_fn("attention_tc", "cml_attn_prefill_tc_maps")(
         _p(q), q.stride(0), _p(out), out.stride(0), _p(k_pages), _p(v_pages), k_pages.shape[0], _p(block_table),
         block_table.shape[1], _p(tile_seq), _p(tile_q0), n_tiles, _p(seq_row0), _p(seq_start), _p(seq_new), n_heads,
         n_kv_heads, head_dim, value_dim, rows_per_tile, heads_per_cta, head_chunks, int(window or 0), float(scale), _p(r1), _p(r2),
         int(chunk or 0), _p(sink), _p(head_gate), head_gate.stride(0) if head_gate is not None else 0, int(gate_col),
-        int(maps), float(softcap or 0.0), 1 if out.dtype == torch.float32 else 0, int(keep_first or 0), _p(err), _stream()),
-        "attn_prefill_tc")
+        int(maps), float(softcap or 0.0), 1 if out.dtype == torch.float32 else 0, int(keep_first or 0), _p(raw_bias),
+        raw_bias.shape[1] if raw_bias is not None else 0, float(out_scale), _p(err), _stream()), "attn_prefill_tc")
 
 
 def maps_difference(maps_out: torch.Tensor, lam: float, eps: float, out_scale: float, out: torch.Tensor, heads: int, value_dim: int):

@@ -8,6 +8,8 @@
 //                                                  o = S^T q / (max(|n . q|, e^(-m')) + 1e-6)
 //
 //   retention (a fixed decay per head):            S <- d S + k v^T;  o = S^T q
+//   state-space recurrence (decay e^(-e^A dt) and step dt per head and token, k and q shared by groups of heads):
+//                                                  S <- e^(-e^A dt) S + dt k v^T;  o = S^T q + D v
 //   generalized delta rule (decay w and removal rate a per key channel, u = k / |k|):
 //                                                  S <- diag(w) S - (a * u)(u^T S) + k v^T;  o = S^T r
 //
@@ -26,6 +28,17 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float logsigmoid_f(float x) { return x < 0.f ? x - log1pf(expf(x)) : -log1pf(expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float split_sum(const float* p, int n, long stride) {
+    float v = p[0];
+    for (int s0 = 1; s0 < n; s0 += 8) {                        // eight splits' loads in flight, added in split order
+        float t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = p[(size_t)min(s0 + k, n - 1) * stride];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += s0 + k < n ? t[k] : 0.f;
+    }
+    return v;
+}
 
 // ------------------------------------------------------------------------------------
 // Short convolution + SiLU (+ unit norm). `proj` [rows, ld] holds, from column 0, the q
@@ -165,6 +178,9 @@ extern "C" int cml_conv_unit(const float* proj, long ld, const float* conv_w, fl
 // column, then n . q, then m after the token.
 // MODE 2, retention. in_a = proj [rows, lda] with q at q_col (heads x D), k at k_col, v at v_col (heads x Dv), q and k
 // turned and scaled already; vec_a [heads]: the heads' decays. state [slots, heads, Dv, D]. out [rows, heads x Dv].
+// MODE 3, state-space recurrence. in_a [rows, lda] from ssm_inputs_kernel: v at v_col (heads x Dv), k and q at k_col and q_col
+// (qk_heads x D, each shared by heads / qk_heads heads); in_b [rows, ldb]: the steps dt (heads), then the decays
+// (heads); vec_a [heads]: D. state [slots, heads, Dv, D]. out [rows, heads x Dv].
 #define SCAN_TOKENS 8
 
 struct ScanParams {
@@ -227,10 +243,10 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
     }
     float m = 0.f;
     if (MODE == 1 && live && !fresh) m = p.state_m[cell];
-    const float keep = MODE == 2 ? p.vec_a[hd] : 0.f;          // retention: the head's decay
-    const int g = MODE == 0 ? hd / (heads / p.qk_heads) : hd;
-    const int qc = MODE == 0 ? g * D : p.q_col + hd * D;
-    const int kc = MODE == 0 ? (p.qk_heads + g) * D : p.k_col + hd * D;
+    const float keep = MODE >= 2 ? p.vec_a[hd] : 0.f;          // retention: the head's decay; state space: its D
+    const int g = (MODE == 0 || MODE == 3) ? hd / (heads / p.qk_heads) : hd;
+    const int qc = MODE == 0 ? g * D : p.q_col + g * D;
+    const int kc = MODE == 0 ? (p.qk_heads + g) * D : p.k_col + g * D;
     const int vc = MODE == 0 ? 2 * p.qk_heads * D + hd * Dv : p.v_col + hd * Dv;
     const float a_rate = (MODE == 0 && !p.decay_ready) ? expf(p.vec_a[hd]) : 0.f;
     const bool head_decay = MODE == 0 && p.decay_dim == 1;      // one decay per head: a number per token (s2), not a row of sg
@@ -269,6 +285,7 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
                 r1 = p.in_b[r * p.ldb + p.b_col + hd];
                 if (head_decay) r2 = p.in_c[r * p.ldc + hd];
             } else if (MODE == 1) { r1 = p.in_a[r * p.lda + p.i_col + hd]; r2 = p.in_a[r * p.lda + p.f_col + hd]; }
+            else if (MODE == 3) { r1 = p.in_b[r * p.ldb + hd]; r2 = p.in_b[r * p.ldb + heads + hd]; }
         }
         // The loads stay here, ahead of the tokens that are worked on meanwhile: without this the compiler moves
         // them down to their first use, where the warp would wait for them. (No instruction is emitted.)
@@ -300,7 +317,7 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
             } else if (MODE == 1) {
                 s1[threadIdx.x] = p.cap * tanhf((r1 + p.vec_a[hd]) / p.cap);
                 s2[threadIdx.x] = logsigmoid_f(p.cap * tanhf((r2 + p.vec_b[hd]) / p.cap));
-            }
+            } else if (MODE == 3) { s1[threadIdx.x] = r1; s2[threadIdx.x] = r2; }
         }
     };
     fetch(0);
@@ -375,22 +392,25 @@ __global__ void __launch_bounds__(128) scan_kernel(const ScanParams p) {
             } else {
                 for (int t = 0; t < nt; ++t) delta_token(t);
             }
-        } else if constexpr (MODE == 2) {
+        } else if constexpr (MODE == 2 || MODE == 3) {
             // Retention, one token: S = d S + k v, then the read-out from the new state; four chains, always in this order.
+            // The state-space recurrence is the same with a decay and a step of the token's own, and D v beside the read-out.
             auto retention_token = [&](int t) {
                 const float* kq = &sk[t][slice * SL];
                 const float* qq = &sq[t][slice * SL];
-                const float vcol = sv[t][wcol];
+                const float raw = sv[t][wcol];
+                const float vcol = MODE == 3 ? raw * s1[t] : raw, fade = MODE == 3 ? s2[t] : keep;
                 float o4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int i = 0; i < DS; i += 4) {
                     const float4 kv = *reinterpret_cast<const float4*>(kq + i), qv = *reinterpret_cast<const float4*>(qq + i);
-                    S[i] = fmaf(keep, S[i], vcol * kv.x); S[i + 1] = fmaf(keep, S[i + 1], vcol * kv.y);
-                    S[i + 2] = fmaf(keep, S[i + 2], vcol * kv.z); S[i + 3] = fmaf(keep, S[i + 3], vcol * kv.w);
+                    S[i] = fmaf(fade, S[i], vcol * kv.x); S[i + 1] = fmaf(fade, S[i + 1], vcol * kv.y);
+                    S[i + 2] = fmaf(fade, S[i + 2], vcol * kv.z); S[i + 3] = fmaf(fade, S[i + 3], vcol * kv.w);
                     o4[0] = fmaf(S[i], qv.x, o4[0]); o4[1] = fmaf(S[i + 1], qv.y, o4[1]);
                     o4[2] = fmaf(S[i + 2], qv.z, o4[2]); o4[3] = fmaf(S[i + 3], qv.w, o4[3]);
                 }
-                const float o = slices_sum<NS>((o4[0] + o4[1]) + (o4[2] + o4[3]));
+                float o = slices_sum<NS>((o4[0] + o4[1]) + (o4[2] + o4[3]));
+                if (MODE == 3) o = fmaf(keep, raw, o);
                 if (live && slice == 0) p.out[(size_t)(row0 + t0 + t) * heads * Dv + hd * Dv + c] = o;
             };
             if (nt == SCAN_TOKENS) {
@@ -500,6 +520,217 @@ extern "C" int cml_retention_scan(const float* proj, long ld, int q_col, int k_c
     return launch_scan<2>(p, n_seqs, (cudaStream_t)stream);
 }
 
+extern "C" int cml_ssm_scan(const float* rows_in, long ld, int x_col, int b_col, int c_col, const float* gates, long ldg,
+                            const float* d_skip, float* state, const int* seq_row0, const int* seq_new, const int* seq_start,
+                            const int* seq_slot, float* out, int n_seqs, int heads, int groups, int D, int Dv, void* stream) {
+    if (groups < 1 || heads % groups) return CML_ERR_BAD_SIZE;
+    ScanParams p = {};
+    p.in_a = rows_in; p.lda = ld; p.in_b = gates; p.ldb = ldg; p.vec_a = d_skip; p.state = state; p.state_m = nullptr;
+    p.seq_row0 = seq_row0; p.seq_new = seq_new; p.seq_start = seq_start; p.seq_slot = seq_slot; p.out = out;
+    p.heads = heads; p.qk_heads = groups; p.D = D; p.Dv = Dv;
+    p.q_col = c_col; p.k_col = b_col; p.v_col = x_col; p.q_scale = 1.0f;
+    return launch_scan<3>(p, n_seqs, (cudaStream_t)stream);
+}
+
+// ------------------------------------------------------------------------------------
+// What the state-space recurrence reads. proj [rows, ld] (n_splits matrices split_stride apart, added in split order):
+// z (inner), then the convolved channels (x, B, C), then one step-size input per head. Every channel passes a causal
+// convolution (conv_w [taps, channels], the last tap the current token's; `state` [slots, max(taps - 1, 1), channels] holds
+// the inputs of the tokens before the step) with bias, then SiLU: out [rows, channels]. The steps: dt = softplus(in +
+// dt_bias), gates [rows, 2 heads] = dt, then exp(-exp(a_log) dt). z_out (may be null) gets z [rows, inner]. With
+// update_state (every sequence of the step brings one row) the state moves on by that row here. A thread takes VEC
+// neighbouring columns of up to `rows_per` rows.
+struct SsmInputs {
+    const float* proj; long ld; int n_splits; long split_stride;
+    const float* conv_w; const float* conv_b; const float* dt_bias; const float* a_log;
+    float* state; int update_state;
+    const int* row_seq; const int* row_pos; const int* seq_row0; const int* seq_slot;
+    float* out; float* gates; float* z_out;
+    int rows, rows_per, inner, channels, heads, taps;
+};
+
+template <int VEC> struct SsmPiece { float v[VEC]; };
+template <int VEC> __device__ __forceinline__ SsmPiece<VEC> ssm_load(const float* p) {
+    SsmPiece<VEC> r;
+    if constexpr (VEC == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w;
+    } else {
+        r.v[0] = p[0];
+    }
+    return r;
+}
+template <int VEC> __device__ __forceinline__ void ssm_store(float* p, const SsmPiece<VEC>& r) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else p[0] = r.v[0];
+}
+template <int VEC> __device__ __forceinline__ SsmPiece<VEC> ssm_sum(const float* p, int n, long stride) {
+    SsmPiece<VEC> r = ssm_load<VEC>(p);
+    for (int s0 = 1; s0 < n; s0 += 8) {                        // eight splits' loads in flight, added in split order
+        SsmPiece<VEC> t[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) t[k] = ssm_load<VEC>(p + (size_t)min(s0 + k, n - 1) * stride);
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+            if (s0 + k < n)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) r.v[e] += t[k].v[e];
+    }
+    return r;
+}
+
+template <int VEC>
+__global__ void __launch_bounds__(128) ssm_inputs_kernel(const SsmInputs p) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int nz = p.z_out ? p.inner / VEC : 0, nc = p.channels / VEC;
+    const int u = blockIdx.x * blockDim.x + threadIdx.x;
+    const int r0 = blockIdx.y * p.rows_per, r1 = min(p.rows, r0 + p.rows_per);
+    if (u >= nc + nz) {                                        // a head's steps and decays
+        const int h = u - nc - nz;
+        if (h >= p.heads) return;
+        const float bias = p.dt_bias[h], rate = expf(p.a_log[h]);
+        for (int r = r0; r < r1; ++r) {
+            const float dt = softplus_f(split_sum(p.proj + (size_t)r * p.ld + p.inner + p.channels + h, p.n_splits, p.split_stride) + bias);
+            p.gates[(size_t)r * 2 * p.heads + h] = dt;
+            p.gates[(size_t)r * 2 * p.heads + p.heads + h] = expf(-rate * dt);
+        }
+        return;
+    }
+    if (u >= nc) {                                             // z
+        const int c = (u - nc) * VEC;
+        for (int r = r0; r < r1; ++r)
+            ssm_store<VEC>(p.z_out + (size_t)r * p.inner + c, ssm_sum<VEC>(p.proj + (size_t)r * p.ld + c, p.n_splits, p.split_stride));
+        return;
+    }
+    const int c = u * VEC, taps = p.taps, keep = max(taps - 1, 1);
+    const float* col = p.proj + p.inner + c;
+    const SsmPiece<VEC> bias = ssm_load<VEC>(p.conv_b + c);
+    SsmPiece<VEC> w[4];                                        // the taps of the token and of the three before it
+#pragma unroll
+    for (int back = 0; back < 4; ++back) w[back] = ssm_load<VEC>(p.conv_w + (size_t)max(taps - 1 - back, 0) * p.channels + c);
+    for (int r = r0; r < r1; ++r) {
+        const int s = p.row_seq[r], pos = p.row_pos[r], inside = r - p.seq_row0[s];
+        float* st = p.state + (size_t)p.seq_slot[s] * keep * p.channels + c;
+        auto input = [&](int back) -> SsmPiece<VEC> {
+            return back <= inside ? ssm_sum<VEC>(col + (size_t)(r - back) * p.ld, p.n_splits, p.split_stride)
+                                  : ssm_load<VEC>(st + (size_t)(taps - 1 + inside - back) * p.channels);
+        };
+        SsmPiece<VEC> acc = bias, own = input(0), before[3];
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            const bool there = k + 1 < taps && k + 1 <= pos;   // (a token before the sequence's start counts as zero)
+            before[k] = there ? input(k + 1) : own;
+            if (!there)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) before[k].v[e] = 0.f;
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+            acc.v[e] = fmaf(w[3].v[e], before[2].v[e], fmaf(w[2].v[e], before[1].v[e], fmaf(w[1].v[e], before[0].v[e], fmaf(w[0].v[e], own.v[e], acc.v[e]))));
+        for (int back = 4; back < taps && back <= pos; ++back) {
+            const SsmPiece<VEC> x = input(back), wb = ssm_load<VEC>(p.conv_w + (size_t)(taps - 1 - back) * p.channels + c);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc.v[e] = fmaf(wb.v[e], x.v[e], acc.v[e]);
+        }
+        if (p.update_state && taps > 1) {
+            for (int j = 0; j + 2 < taps; ++j) {
+                SsmPiece<VEC> t = ssm_load<VEC>(st + (size_t)(j + 1) * p.channels);
+                if (pos + j + 2 < taps)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) t.v[e] = 0.f;
+                ssm_store<VEC>(st + (size_t)j * p.channels, t);
+            }
+            ssm_store<VEC>(st + (size_t)(taps - 2) * p.channels, own);
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc.v[e] = silu_f(acc.v[e]);
+        ssm_store<VEC>(p.out + (size_t)r * p.channels + c, acc);
+    }
+}
+
+extern "C" int cml_ssm_inputs(const float* proj, long ld, int n_splits, long split_stride, const float* conv_w, const float* conv_b,
+                              const float* dt_bias, const float* a_log, float* state, int update_state, const int* row_seq,
+                              const int* row_pos, const int* seq_row0, const int* seq_slot, float* out, float* gates, float* z_out,
+                              int rows, int inner, int channels, int heads, int taps, void* stream) {
+    if (rows <= 0) return 0;
+    if (n_splits < 1 || inner < 1 || channels < 1 || heads < 1 || taps < 1) return CML_ERR_BAD_SIZE;
+    SsmInputs p = {proj, ld, n_splits, split_stride, conv_w, conv_b, dt_bias, a_log, state, update_state, row_seq, row_pos, seq_row0,
+                   seq_slot, out, gates, z_out, rows, 1, inner, channels, heads, taps};
+    const bool vec = (((long)inner | (long)channels | ld | split_stride) & 3) == 0 &&
+                     ((((uintptr_t)proj) | ((uintptr_t)conv_w) | ((uintptr_t)conv_b) | ((uintptr_t)state) | ((uintptr_t)out) | ((uintptr_t)z_out)) & 15) == 0;
+    const int per = vec ? 4 : 1;
+    const long units = (long)channels / per + (z_out ? inner / per : 0) + heads;
+    if (!update_state && rows > 256) p.rows_per = 8;           // prompts: a thread's taps serve several rows
+    if (((long)rows + p.rows_per - 1) / p.rows_per > 65535) p.rows_per = (int)((rows + 65534L) / 65535);
+    const dim3 grid((unsigned)((units + 127) / 128), (unsigned)((rows + p.rows_per - 1) / p.rows_per));
+    if (vec) launch_pdl(ssm_inputs_kernel<4>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+    else launch_pdl(ssm_inputs_kernel<1>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+    return cml_launch_status();
+}
+
+// After the state-space scan: v = y * silu(z), a row's `groups` equal parts each divided by its own root mean square
+// (eps inside), times w, in the compute type. y [rows, width] float; z [rows, ldz] float; w [width] float; out rows ldo
+// apart. A block owns one (row, part), whose values stay in shared memory between the two passes.
+template <typename TO>
+__global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, long ldz,
+                                                               const float* __restrict__ w, TO* __restrict__ out, long ldo, int width,
+                                                               int part, float eps) {
+    extern __shared__ __align__(16) float gg_row[];
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = blockIdx.x, c0 = blockIdx.y * part;
+    const float* yr = y + (size_t)r * width + c0;
+    const float* zr = z + (size_t)r * ldz + c0;
+    float ss = 0.f;
+    const bool vec = (((long)part | (long)width | ldz) & 3) == 0 && ((((uintptr_t)y) | ((uintptr_t)z)) & 15) == 0;
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < part; c += blockDim.x * 4) {
+            const float4 a = *reinterpret_cast<const float4*>(yr + c), g = *reinterpret_cast<const float4*>(zr + c);
+            const float4 v = make_float4(a.x * silu_f(g.x), a.y * silu_f(g.y), a.z * silu_f(g.z), a.w * silu_f(g.w));
+            *reinterpret_cast<float4*>(gg_row + c) = v;
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+    } else {
+        for (int c = threadIdx.x; c < part; c += blockDim.x) {
+            const float v = yr[c] * silu_f(zr[c]);
+            gg_row[c] = v;
+            ss = fmaf(v, v, ss);
+        }
+    }
+    const float scale = 1.0f / sqrtf(block_sum(ss, red) / (float)part + eps);
+    TO* o = out + (size_t)r * ldo + c0;
+    if (vec) {                                                 // each thread reads back what it wrote itself
+        for (int c = threadIdx.x * 4; c < part; c += blockDim.x * 4)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[c + e] = from_f32<TO>(gg_row[c + e] * scale * w[c0 + c + e]);
+    } else {
+        for (int c = threadIdx.x; c < part; c += blockDim.x) o[c] = from_f32<TO>(gg_row[c] * scale * w[c0 + c]);
+    }
+}
+
+extern "C" int cml_gated_group_norm(const float* y, const float* z, long ldz, const float* w, void* out, long ldo, int out_dtype, int rows,
+                                    int width, int groups, float eps, void* stream) {
+    if (rows <= 0) return 0;
+    if (groups < 1 || groups > 65535 || width % groups) return CML_ERR_BAD_SIZE;
+    const int part = width / groups;
+    const size_t smem = (size_t)part * sizeof(float);
+    if (smem > 200 * 1024) return CML_ERR_BAD_SIZE;
+    const int block = part >= 1024 ? 256 : part >= 256 ? 128 : part >= 64 ? 64 : 32;
+#define GG_CASE(T_, D_)                                                                                                   \
+    if (out_dtype == D_) {                                                                                                \
+        if (smem > 48 * 1024 && cml_allow_smem<gated_group_norm_kernel<T_>>(smem) != cudaSuccess) return CML_ERR_BAD_SIZE; \
+        launch_pdl(gated_group_norm_kernel<T_>, dim3(rows, groups), dim3(block), smem, (cudaStream_t)stream, y, z, ldz, w, \
+                   (T_*)out, ldo, width, part, eps);                                                                      \
+        return cml_launch_status();                                                                                       \
+    }
+    GG_CASE(float, CML_DTYPE_F32)
+    GG_CASE(bf16, CML_DTYPE_BF16)
+#undef GG_CASE
+    return CML_ERR_BAD_DTYPE;
+}
+
 // ------------------------------------------------------------------------------------
 // Generalized delta rule. Both terms of the write read the old state, so with p = k^T S (S before the token), q = (r * w)^T S,
 // n2 = 1 / (sum k^2 + 1e-6) the token is
@@ -524,18 +755,6 @@ struct DeltaInputs {
     float* packed; float* scal; float* gate_out;
     int heads, D, Dv;
 };
-
-__device__ __forceinline__ float split_sum(const float* p, int n, long stride) {
-    float v = p[0];
-    for (int s0 = 1; s0 < n; s0 += 8) {                        // eight splits' loads in flight, added in split order
-        float t[8];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) t[k] = p[(size_t)min(s0 + k, n - 1) * stride];
-#pragma unroll
-        for (int k = 0; k < 8; ++k) v += s0 + k < n ? t[k] : 0.f;
-    }
-    return v;
-}
 
 template <typename T>
 __global__ void __launch_bounds__(256) delta_inputs_kernel(const DeltaInputs p) {

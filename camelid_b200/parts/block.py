@@ -150,6 +150,8 @@ class PostNormBlock(Part):
     next reader. A layer without a feed-forward has only the first sublayer. ``after``: a part that runs at the end of
     the layer (a per-layer token input)."""
 
+    norm_entry = "sum_normed"               # what the arrangement asks of its norms
+
     def __init__(self, layer_spec):
         super().__init__({}, "")
         from ..errors import ConfigError
@@ -160,14 +162,14 @@ class PostNormBlock(Part):
         self.norm2 = build_part("norm", layer_spec.norm2) if self.ffn is not None else None
         self.after = build_part("layer_input", layer_spec.after) if layer_spec.after is not None else None
         if self.ffn is not None and layer_spec.norm2 is None:
-            raise ConfigError("block.arrangement", "the postnorm arrangement needs norm2 with a feed-forward")
+            raise ConfigError("block.arrangement", f"the {self.kind} arrangement needs norm2 with a feed-forward")
         if not hasattr(self.mixer, "branch_output"):
             raise ConfigError("mixer.kind", f"the mixer {self.mixer.kind!r} does not hand its output over (branch_output)")
         if self.ffn is not None and not hasattr(self.ffn, "output"):
             raise ConfigError("ffn.kind", f"the feed-forward {self.ffn.kind!r} does not hand its output over (output)")
         for n in (self.norm1, self.norm2):
-            if n is not None and not hasattr(n, "sum_normed"):
-                raise ConfigError("norm.kind", f"the norm {n.kind!r} cannot norm a residual sum in place (sum_normed)")
+            if n is not None and not hasattr(n, self.norm_entry):
+                raise ConfigError("norm.kind", f"the norm {n.kind!r} cannot stand behind a sublayer here ({self.norm_entry})")
 
     def parts(self):
         return tuple(p for p in (self.norm1, self.mixer, self.norm2, self.ffn, self.after) if p is not None)
@@ -205,6 +207,25 @@ class PostNormBlock(Part):
             y, bias = self.ffn.output(ctx, x, "ffn_out", stream=h) if getattr(self.ffn, "takes_stream", False) \
                 else self.ffn.output(ctx, x, "ffn_out")
             x = self.norm2.sum_normed(ctx, y, h, self.alpha, bias)
+        if self.after is not None:
+            self.after.forward(ctx, x, h)
+
+
+@register_part("block", "outnorm")
+class OutputNormBlock(PostNormBlock):
+    """Only the sublayers' outputs are normed: x += s * norm1(mixer(x)), then x += s * norm2(ffn(x)), s one number of the layer
+    (``residual_scale``). The sublayers read x as it is and hand their output over as in ``postnorm``; the norm adds and
+    leaves the new rows in the compute type in one pass (``add_normed_rows``)."""
+    norm_entry = "add_normed_rows"
+
+    def forward(self, ctx, h):
+        ctx.settle(h)                       # whatever a layer of another arrangement left undone
+        x = ctx.stream_rows(h)
+        x = self.norm1.add_normed_rows(ctx, self.mixer.branch_output(ctx, x, "mixer_out"), h, self.alpha)
+        if self.ffn is not None:
+            y, bias = self.ffn.output(ctx, x, "ffn_out", stream=h) if getattr(self.ffn, "takes_stream", False) \
+                else self.ffn.output(ctx, x, "ffn_out")
+            x = self.norm2.add_normed_rows(ctx, y, h, self.alpha, bias)
         if self.after is not None:
             self.after.forward(ctx, x, h)
 

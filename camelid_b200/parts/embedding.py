@@ -14,7 +14,8 @@ from .base import Part, TensorSpec, register_part, to_device
 class TokenEmbedding(Part):
     """x = scale * E[token] (+ P[position]). ``scale`` (default 1) multiplies the embedding row; ``position_tensor``
     names a table of learned position rows [``positions``, hidden] that are added unscaled (positions count from 0 in
-    every sequence; the plan's ``max_position`` keeps sequences inside the table)."""
+    every sequence; the plan's ``max_position`` keeps sequences inside the table). ``stream_rows``: the first layer reads the
+    stream as it is, so its rows are written in the compute type too."""
     graph_safe = True
     graph_safe_any_step = True
 
@@ -26,6 +27,7 @@ class TokenEmbedding(Part):
         self.scale = float(params["scale"]) if params.get("scale") is not None else 1.0
         self.position_tensor = params.get("position_tensor")
         self.positions = int(params["positions"]) if self.position_tensor else 0
+        self.stream_rows = bool(params.get("stream_rows", False))
         self.weight = None
         self.position_rows = None
 
@@ -41,7 +43,7 @@ class TokenEmbedding(Part):
             self.position_rows = to_device(tensors[self.position_tensor], device, dtype)
 
     def forward(self, ctx, tokens, out, err):
-        if self.scale == 1.0 and self.position_rows is None:
+        if self.scale == 1.0 and self.position_rows is None and not (self.stream_rows and ctx.dtype != torch.float32):
             ops.embed_gather(self.weight, tokens, out, err)
             return
         # the same rows in the compute type too: a first layer that reads the stream as it is needs no pass of its own

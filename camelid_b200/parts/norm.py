@@ -85,3 +85,11 @@ class RMSNorm(Part):
         ops.post_norm_add(y, bias, self.weight, self.eps, scale, residual, then.weight if fuse else None,
                           then.eps if fuse else 0.0, x)
         return x
+
+    def add_normed_rows(self, ctx, y, residual, scale: float = 1.0, bias=None):
+        """residual += scale * rmsnorm(y + bias) * w, and the stream's new rows in the compute type (the stream itself on the
+        float32 path) for parts that read the stream as it is; one pass."""
+        x = ctx.buffer("stream_rows", residual.shape) if ctx.dtype != torch.float32 else None
+        ops.post_norm_add(y, bias, self.weight, self.eps, scale, residual, None, 0.0, x)
+        ctx.rows_copy = (residual, x) if x is not None else None
+        return x if x is not None else residual

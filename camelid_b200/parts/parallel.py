@@ -6,6 +6,10 @@ outputs, each first RMS-normed over the model width with a weight of its own
 
 A branch is any registered mixer that offers ``branch_output(ctx, x, name)``; each keeps its
 own cache or state (the entry's cache needs are the branches' together).
+
+With ``scales`` (a number per branch) the layer's output is the weighted sum of the branches' instead, without norms or
+tensors of its own:  y = sum over b of scales[b] * mixer_b(x).  The branches' rows then stand side by side, each times its
+scale (``output_rows``, ``scale_output``), and one product with their output matrices side by side makes the sum.
 """
 from __future__ import annotations
 
@@ -29,7 +33,14 @@ class ParallelMixers(Part):
         for name, b in zip(self.names, self.branches):
             if not hasattr(b, "branch_output"):
                 raise ConfigError("branches", f"the mixer {b.kind!r} of branch {name!r} cannot stand beside others")
-        self.out_w = None
+        self.scales = tuple(float(c) for c in params["scales"]) if params.get("scales") is not None else None
+        if self.scales is not None:
+            if len(self.scales) != len(self.branches):
+                raise ConfigError("scales", f"one number per branch: {len(self.branches)} branches, {len(self.scales)} numbers")
+            for name, b in zip(self.names, self.branches):
+                if not (hasattr(b, "output_rows") and hasattr(b, "scale_output")):
+                    raise ConfigError("branches", f"the mixer {b.kind!r} of branch {name!r} cannot enter a weighted sum")
+        self.out_w = self.w_joint = None
 
     @property
     def graph_safe(self):
@@ -43,26 +54,39 @@ class ParallelMixers(Part):
         specs = {}
         for name, b in zip(self.names, self.branches):
             specs.update(b.tensor_specs())
-            specs[f"{self.prefix}{name}.out"] = TensorSpec((self.hidden_size,), "norm")
+            if self.scales is None:
+                specs[f"{self.prefix}{name}.out"] = TensorSpec((self.hidden_size,), "norm")
         return specs
 
     def load(self, tensors, device, dtype):
         for b in self.branches:
             b.load(tensors, device, dtype)
-        self.out_w = [tensors[f"{self.prefix}{name}.out"].to(device=device, dtype=torch.float32).contiguous()
-                      for name in self.names]
+        if self.scales is None:
+            self.out_w = [tensors[f"{self.prefix}{name}.out"].to(device=device, dtype=torch.float32).contiguous()
+                          for name in self.names]
+        else:                           # the output matrices' columns side by side; each branch keeps its own as a view
+            self.w_joint = torch.cat([b.output_weight() for b in self.branches], dim=1).contiguous()
+            at = 0
+            for b, c in zip(self.branches, self.scales):
+                k = b.output_weight().shape[1]
+                b.set_output_weight(self.w_joint[:, at:at + k])
+                b.scale_output(c)
+                at += k
         # Branches that read the same rows through one stacked input matrix each (``w_in``): all of them stacked
         # once more, so that one product serves every branch; each keeps its rows of it as a view.
         self.w_in = None
         self.in_cols = []
         if len(self.branches) > 1 and all(getattr(b, "w_in", None) is not None for b in self.branches):
-            stacked = torch.cat([b.w_in for b in self.branches], dim=0).contiguous()
+            # (each branch's rows padded to a multiple of 8 with zeros: its columns of the product start on 16 bytes)
+            padded = [-b.w_in.shape[0] % 8 for b in self.branches]
+            pieces = [t for b, pad in zip(self.branches, padded) for t in ([b.w_in, b.w_in.new_zeros((pad, b.w_in.shape[1]))] if pad else [b.w_in])]
+            stacked = torch.cat(pieces, dim=0).contiguous()
             at = 0
-            for b in self.branches:
+            for b, pad in zip(self.branches, padded):
                 n = b.w_in.shape[0]
                 b.w_in = stacked[at:at + n]
                 self.in_cols.append((at, n))
-                at += n
+                at += n + pad
             self.w_in = stacked
 
     def cache_spec(self):
@@ -71,12 +95,37 @@ class ParallelMixers(Part):
     def query_tile_sizes(self):
         return [r for b in self.branches for r in b.query_tile_sizes()]
 
+    def _projections(self, ctx, x):
+        """Every branch's columns of the stacked input product (None each where there is no such product): complete rows, or
+        split sums on one-token steps where every branch takes those."""
+        if self.w_in is None:
+            return [None] * len(self.branches)
+        from . import linear
+        split = ctx.decode and all(getattr(b, "takes_split_rows", False) for b in self.branches)
+        proj = (linear.product_f32 if split else linear.product_rows_f32)(ctx, x, self.w_in, "branches_proj")
+        return [proj[..., at:at + n] for at, n in self.in_cols]
+
+    def _joint_rows(self, ctx, x):
+        rows = ctx.buffer("branches_rows", (ctx.n_rows, self.w_joint.shape[1]))
+        at = 0
+        for b, proj in zip(self.branches, self._projections(ctx, x)):
+            k = b.output_weight().shape[1]
+            b.output_rows(ctx, x, rows[:, at:at + k], proj)
+            at += k
+        return rows
+
     def forward(self, ctx, x, residual):
-        if self.w_in is not None:
+        if self.w_joint is not None:
             from . import linear
-            proj = linear.product_rows_f32(ctx, x, self.w_in, "branches_proj")
-            ys = [b.branch_output(ctx, x, f"branch{i}_out", proj[:, at:at + n])
-                  for i, (b, (at, n)) in enumerate(zip(self.branches, self.in_cols))]
-        else:
-            ys = [b.branch_output(ctx, x, f"branch{i}_out") for i, b in enumerate(self.branches)]
+            linear.add_into_residual(ctx, self._joint_rows(ctx, x), self.w_joint, residual, "o_partial")
+            return
+        ys = [b.branch_output(ctx, x, f"branch{i}_out", proj) if proj is not None else b.branch_output(ctx, x, f"branch{i}_out")
+              for i, (b, proj) in enumerate(zip(self.branches, self._projections(ctx, x)))]
         ops.norm_combine(list(zip(ys, self.out_w)), residual, self.eps, 1.0 / len(self.branches))
+
+    def branch_output(self, ctx, x, name: str):
+        """The weighted sum as float32 rows or split sums, for a block that norms it before it is added."""
+        from . import linear
+        if self.w_joint is None:
+            raise ConfigError("branches", "branches whose outputs are normed one by one add into the stream themselves")
+        return linear.product_f32(ctx, self._joint_rows(ctx, x), self.w_joint, name)

@@ -8,7 +8,7 @@ Frequencies as the reference computes them, in float32: f_i = theta^(-2i / rotar
 (src/inference/rope.rs:526-537), then for ``llama3`` scaling: wavelength = 2 pi / f; below
 original/high the frequency stays, above original/low it is divided by the factor, between
 them it is blended with smooth = (original / wavelength - low) / (high - low)
-(src/inference/rope.rs:687-711). ``ramp`` scaling (the YaRN law): with dims = rotary_dim and
+(src/inference/rope.rs:687-711). ``linear`` scaling divides every frequency by the factor. ``ramp`` scaling (the YaRN law): with dims = rotary_dim and
 where(t) = dims ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1)
 and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency is f_i / factor * r_i + f_i (1 - r_i), and sines and
 cosines are multiplied by the ``amplitude`` 0.1 ln(factor) + 1, which the mixer's kernel applies."""
@@ -40,6 +40,8 @@ def rotary_frequencies(rotary_dim: int, theta: float, scaling: dict | None) -> n
             blended = ((f32(1.0) - smooth) * freq / factor + smooth * freq).astype(np.float32)
             freq = np.where(wavelength < orig / high, freq,
                             np.where(wavelength > orig / low, (freq / factor).astype(np.float32), blended)).astype(np.float32)
+        elif kind == "linear":
+            freq = (np.float64(theta) ** (-2.0 * np.arange(rotary_dim // 2, dtype=np.float64) / rotary_dim) / float(scaling["factor"])).astype(np.float32)
         elif kind == "ramp":
             factor, orig = float(scaling["factor"]), float(scaling["original"])
             where = lambda turns: rotary_dim * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))   # noqa: E731

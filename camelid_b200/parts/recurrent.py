@@ -304,6 +304,109 @@ class Retention(Part):
         return linear.product_f32(ctx, self.read_out(ctx, x), self.w_o, name)
 
 
+@register_part("mixer", "state_space")
+class StateSpace(Part):
+    """The state-space recurrence with one decay per head and token (Mamba-2). One input product gives, in this order, z (``inner`` =
+    ``num_heads`` x ``value_dim``), x (``inner``), B and C (``groups`` x ``state_size`` each) and one step-size input per head. x, B and C
+    together pass a short causal convolution per channel (``conv`` [channels, taps], the last tap the current token's, bias
+    ``conv.b``) and SiLU; dt = softplus(input + ``dt_bias``). Per head (which shares B and C with the others of its group)
+
+        S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T,   y_t = S_t^T C_t + D x_t
+
+    y times silu(z), the row's ``norm_groups`` equal parts each divided by its own root mean square, times ``norm``, is projected by
+    ``o``. S (float32, zero at the start) and the convolution's last taps - 1 inputs are the sequence's state; steps, decays,
+    the recurrence and the norm are float32. Tensors ``in conv conv.b dt_bias A_log D norm o``."""
+    graph_safe = True
+    graph_safe_any_step = True
+    takes_split_rows = True                 # the input product's rows may come as split sums
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.hidden_size = int(params["hidden_size"])
+        self.eps = float(params.get("eps", 1e-6))
+        self.num_heads = int(params["num_heads"])
+        self.value_dim = int(params["value_dim"])
+        self.state_size = int(params["state_size"])
+        self.groups = int(params.get("groups") or 1)
+        self.norm_groups = int(params.get("norm_groups") or 1)
+        self.taps = int(params["conv_taps"])
+        if not 1 <= self.state_size <= 256:
+            raise ConfigError("state_size", f"the scan kernels take states of 1..256 channels, got {self.state_size}")
+        _check_dims(self.state_size, self.value_dim)
+        self.inner = self.num_heads * self.value_dim
+        if self.groups <= 0 or self.num_heads % self.groups:
+            raise ConfigError("groups", f"{self.groups} groups do not divide {self.num_heads} heads")
+        if self.norm_groups <= 0 or self.inner % self.norm_groups:
+            raise ConfigError("norm_groups", f"{self.norm_groups} parts do not divide {self.inner} channels")
+        if self.taps < 1:
+            raise ConfigError("conv_taps", f"must be at least 1, got {self.taps}")
+        self.channels = self.inner + 2 * self.groups * self.state_size         # x, B, C
+        self.cols = (0, self.inner, self.inner + self.groups * self.state_size)
+        self.in_width = self.inner + self.channels + self.num_heads
+        self.w_in = self.w_o = self.conv_w = self.conv_b = self.dt_bias = self.a_log = self.d_skip = self.norm_w = None
+
+    def tensor_specs(self):
+        p, hid, h = self.prefix, self.hidden_size, self.num_heads
+        return {p + "in": TensorSpec((self.in_width, hid)), p + "conv": TensorSpec((self.channels, self.taps), "conv"),
+                p + "conv.b": TensorSpec((self.channels,), "input_bias"), p + "dt_bias": TensorSpec((h,), "log_rate"),
+                p + "A_log": TensorSpec((h,), "log_rate"), p + "D": TensorSpec((h,), "norm"), p + "norm": TensorSpec((self.inner,), "norm"),
+                p + "o": TensorSpec((hid, self.inner))}
+
+    def load(self, tensors, device, dtype):
+        p = self.prefix
+        f32 = lambda n: tensors[p + n].to(device=device, dtype=torch.float32).contiguous()      # noqa: E731
+        w = to_device(tensors[p + "in"], device, dtype)
+        pad = -w.shape[0] % 8                       # rows of zeros, so that the product's float rows start on 16 bytes
+        self.w_in = torch.cat([w, w.new_zeros((pad, w.shape[1]))], 0).contiguous() if pad else w
+        self.w_o = to_device(tensors[p + "o"], device, dtype)
+        self.conv_w = f32("conv").t().contiguous()  # tap by tap: the channels of a tap side by side
+        self.conv_b, self.dt_bias, self.a_log, self.d_skip, self.norm_w = f32("conv.b"), f32("dt_bias"), f32("A_log"), f32("D"), f32("norm")
+
+    def cache_spec(self):
+        return [StateSpec((self.num_heads, self.value_dim, self.state_size), "float32", "ssm"),
+                StateSpec((max(self.taps - 1, 1), self.channels), "float32", "ssm_conv")]
+
+    def read_out(self, ctx, x, out=None, proj=None):
+        n, H = ctx.n_rows, self.num_heads
+        if proj is None:                            # (the kept inputs of a step of several rows per sequence are read from complete rows)
+            proj = (linear.product_f32 if ctx.decode else linear.product_rows_f32)(ctx, x, self.w_in, "ss_proj")
+        z = ctx.buffer("ss_z", (n, self.inner), torch.float32) if proj.dim() == 3 else None
+        rows = ctx.buffer("ss_rows", (n, self.channels), torch.float32)
+        gates = ctx.buffer("ss_gates", (n, 2 * H), torch.float32)
+        conv_state = ctx.state("ssm_conv")
+        ops.ssm_inputs(proj, self.conv_w, self.conv_b, self.dt_bias, self.a_log, conv_state, ctx.row_seq, ctx.row_pos, ctx.seq_row0,
+                       ctx.seq_slot, rows, gates, self.inner, z, update_state=ctx.decode)
+        if self.taps > 1 and not ctx.decode:
+            ops.keep_last_rows(proj, self.inner, self.channels, conv_state, ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot,
+                               ctx.n_seqs)
+        y = ctx.buffer("ss_y", (n, self.inner), torch.float32)
+        ops.ssm_scan(rows, self.cols, gates, self.d_skip, ctx.state("ssm"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, y,
+                     ctx.n_seqs, H, self.groups, self.state_size, self.value_dim)
+        if out is None:
+            out = ctx.buffer("ss_out", (n, self.inner))
+        ops.gated_group_norm(y, z if z is not None else proj[:, :self.inner], self.norm_w, self.norm_groups, self.eps, out)
+        return out
+
+    def forward(self, ctx, x, residual):
+        linear.add_into_residual(ctx, self.read_out(ctx, x), self.w_o, residual, "o_partial")
+
+    def branch_output(self, ctx, x, name: str, proj=None):
+        return linear.product_f32(ctx, self.read_out(ctx, x, None, proj), self.w_o, name)
+
+    # a parent may put the rows that go into ``o`` beside others', with a factor of its own, and run one product for all
+    def output_weight(self):
+        return self.w_o
+
+    def set_output_weight(self, w):
+        self.w_o = w
+
+    def output_rows(self, ctx, x, out, proj=None):
+        self.read_out(ctx, x, out, proj)
+
+    def scale_output(self, factor: float):
+        self.norm_w = self.norm_w * float(factor)
+
+
 @register_part("mixer", "general_delta")
 class GeneralDelta(Part):
     """The delta rule with a decay w and a removal rate a per key channel. r, k (``num_heads`` x ``key_dim``) and v
