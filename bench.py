@@ -12,7 +12,8 @@ Nudusun decoder (differential window attention and gated delta layers, routed fe
 of equal size, ``--kizezen small,medium`` for the Kizezen decoder (retention, windowed attention with kept first keys and
 attention over a latent in turn, dense feed-forwards) beside the Zulozen decoder of equal size, ``--ramopel small,medium``
 for the Ramopel decoder (windowed attention over a latent and the generalized delta rule in turn, dense and routed
-feed-forwards) beside the Kizezen decoder of equal size.
+feed-forwards) beside the Kizezen decoder of equal size, ``--zabunex small,medium`` for the Zabunex decoder (attention beside a
+state-space recurrence and attention with a bias by distance in turn) beside the Kizezen decoder of equal size.
 This library runs on one GPU: for --gpus above 1 it says so and exits with 2."""
 import argparse
 import json
@@ -54,6 +55,9 @@ def main() -> int:
     ap.add_argument("--ramopel", default=None, metavar="SIZES",
                     help="instead of the default workload: decode and prefill of the Ramopel decoder beside the Kizezen "
                          "decoder of equal size, e.g. small,medium,wide (prompts of 512 tokens, --batch, --steps)")
+    ap.add_argument("--zabunex", default=None, metavar="SIZES",
+                    help="instead of the default workload: decode and prefill of the Zabunex decoder beside the Kizezen "
+                         "decoder of equal size, e.g. small,medium,wide (prompts of 512 tokens, --batch, --steps)")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}))
@@ -81,6 +85,10 @@ def main() -> int:
         return 0
     if args.ramopel:
         print(json.dumps(benchmark.run_ramopel(tuple(args.ramopel.split(",")), batch=args.batch, steps=min(args.steps, 64),
+                                               warmup=max(min(args.warmup, 8), 3), dtype=args.dtype)))
+        return 0
+    if args.zabunex:
+        print(json.dumps(benchmark.run_zabunex(tuple(args.zabunex.split(",")), batch=args.batch, steps=min(args.steps, 64),
                                                warmup=max(min(args.warmup, 8), 3), dtype=args.dtype)))
         return 0
     rec = benchmark.run(batch=args.batch, prompt_tokens=args.prompt_tokens, decode_steps=args.steps,

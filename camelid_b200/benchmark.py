@@ -1048,6 +1048,135 @@ def run_ramopel(sizes=("small", "medium"), batch: int = 8, prompt_tokens: int = 
     return out
 
 
+ZABUNEX_SIZES = {
+    # width, layers (the parallel mixer and attention over all earlier keys, in turn), feed-forward size, query and kv heads of
+    # `head` channels in both attentions, blocks of positions of the parallel one, the state-space half's heads of `ssm_head`
+    # channels, its state and groups, rows and reach of the bias by distance
+    "small": dict(width=1024, layers=8, ff=4096, heads=8, kv_heads=2, head=128, block=512, ssm_heads=32, ssm_head=64, state=128, groups=4,
+                  bias_rows=32, bias_max=256, vocab=32768),
+    "medium": dict(width=2048, layers=16, ff=8192, heads=16, kv_heads=4, head=128, block=1024, ssm_heads=64, ssm_head=64, state=128,
+                   groups=8, bias_rows=32, bias_max=256, vocab=32768),
+    "wide": dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, head=128, block=1024, ssm_heads=128, ssm_head=64, state=128,
+                 groups=8, bias_rows=32, bias_max=256, vocab=32768),
+}
+
+
+def zabunex_config_for(size: str) -> dict:
+    s = ZABUNEX_SIZES[size]
+    heads = {"dim": s["head"], "vdim": s["head"], "heads": s["heads"], "kv_heads": s["kv_heads"], "scale": s["head"] ** -0.5}
+    attention = {**heads, "bias_max": s["bias_max"], "bias_rows": s["bias_rows"], "q_temp": {"coef": 0.1, "every": 4096}}
+    left = {**heads, "conv": 4, "mask": {"size": s["block"]}, "rot": {"dims": s["head"] // 2, "base": 500000.0, "scaling": {"factor": 2.0}}}
+    right = {"heads": s["ssm_heads"], "vdim": s["ssm_head"], "state": s["state"], "groups": s["groups"], "norm_groups": s["groups"], "conv": 4}
+    kinds = (("parallel", {"left": left, "right": right, "left_scale": 0.5, "right_scale": 0.5}), ("attention", attention))
+    layers = [{"type": kinds[i % 2][0], "mixer": copy.deepcopy(kinds[i % 2][1]), "mlp": {"kind": "dense", "ff": s["ff"]}}
+              for i in range(s["layers"])]
+    return {"architecture": "Zabunex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
+def kizezen_config_like_zabunex(size: str) -> dict:
+    """The Kizezen decoder of the same width, depth, attention heads and vocabulary, retention and attention over all earlier keys in
+    turn (the library's closest model: grouped attention with norms over the whole projections and a sink, a matrix state per
+    head), dense feed-forwards; each as large as makes a layer's matrices hold as many elements as the other's."""
+    s = ZABUNEX_SIZES[size]
+    H, D, W = s["heads"], s["head"], s["width"]
+    attention = {"dim": D, "vdim": D, "heads": H, "kv_heads": s["kv_heads"], "scale": D ** -0.5, "rot": {"dims": D, "base": 10000.0}}
+    retention = {"dim": D, "vdim": D, "heads": H, "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * i / max(H - 1, 1)) for i in range(H)],
+                 "rot": {"dims": D, "base": 10000.0}}
+    layers = []
+    for i, L in enumerate(zabunex_config_for(size)["layers"]):
+        kind, mixer = (("attention", attention) if L["type"] == "attention" else ("retention", retention))
+        mine = {"type": kind, "mixer": dict(mixer), "mlp": None}
+        ff = (_zabunex_matrices(L, W) - _kizezen_matrices(mine, W)) // (2 * W) // 64 * 64
+        layers.append({**mine, "mlp": {"kind": "dense", "ff": int(ff)}})
+    return {"architecture": "Kizezen", "vocab": s["vocab"], "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_scale": 1.0, "layers": layers}
+
+
+def _zabunex_matrices(L: dict, W: int) -> float:
+    """Elements of the matrices a row passes in one layer."""
+    m, f = L["mixer"], L.get("mlp")
+    if L["type"] == "attention":
+        n = W * m["dim"] * (2 * m["heads"] + m["kv_heads"])
+    else:
+        a, b = m["left"], m["right"]
+        inner = b["heads"] * b["vdim"]
+        n = W * (a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"]) + a["heads"] * a["vdim"])
+        n += W * (3 * inner + 2 * b["groups"] * b["state"] + b["heads"])
+    return n + (2 * W * f["ff"] if f else 0)
+
+
+def zabunex_step_bytes(cfg: dict, batch: int, context: float, elem: int) -> dict:
+    """Bytes a decode step must move: every matrix once (the output head, no embedding table), the keys and values a query
+    sees (of the blocks of positions half a block on average), every state-space state read and written in float32."""
+    W = cfg["width"]
+    weights = kv = state = 0.0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        weights += _zabunex_matrices(L, W)
+        a = m if L["type"] == "attention" else m["left"]
+        seen = context
+        if a.get("mask"):
+            seen = min(context, a["mask"]["size"]) if context <= a["mask"]["size"] else a["mask"]["size"] / 2
+        kv += batch * seen * a["kv_heads"] * (a["dim"] + a["vdim"])
+        if L["type"] == "parallel":
+            b = m["right"]
+            state += 2.0 * batch * b["heads"] * b["vdim"] * b["state"] * 4
+    weights += cfg["vocab"] * W
+    return {"weights": int(weights * elem), "kv": int(kv * elem), "state": int(state), "total": int((weights + kv) * elem + state)}
+
+
+def zabunex_prefill_flops(cfg: dict, tokens: int) -> float:
+    """2 x tokens x (elements of every matrix a token passes) plus the attention over the visible keys (per head and pair of
+    positions the key's and the value's channels) and 4 flops per element of a state-space state and token."""
+    W = cfg["width"]
+    total = 0.0
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        total += 2.0 * tokens * _zabunex_matrices(L, W)
+        a = m if L["type"] == "attention" else m["left"]
+        block = a["mask"]["size"] if a.get("mask") else tokens
+        total += 2.0 * sum(i % block + 1 for i in range(tokens)) * a["heads"] * (a["dim"] + a["vdim"])
+        if L["type"] == "parallel":
+            b = m["right"]
+            total += 4.0 * tokens * b["heads"] * b["vdim"] * b["state"]
+    return total + 2.0 * W * cfg["vocab"]
+
+
+def run_zabunex(sizes=("small", "medium"), batch: int = 8, prompt_tokens: int = 512, steps: int = 64, warmup: int = 4,
+                prefill_tokens: int = 2048, dtype: str = "bfloat16") -> dict:
+    """Decode steps (timed on the device in the loop ``generate`` runs) and prefill steps of the Zabunex decoder and of
+    the Kizezen decoder of equal width, depth, heads and vocabulary, random weights."""
+    from . import api
+    pk = peaks()
+    elem = 2 if dtype == "bfloat16" else 4
+    out = {"metric": "decode and prefill tokens/s, Zabunex beside the Kizezen decoder of equal size", "dtype": dtype,
+           "batch": batch, "prompt_tokens": prompt_tokens, "steps": steps, "warmup": warmup,
+           "prefill_tokens": prefill_tokens, "peaks": pk["source"], "data": "synthetic (seeded uniform token ids, random weights)",
+           "sizes": {}}
+    for size in sizes:
+        rec = {"shape": ZABUNEX_SIZES[size]}
+        for label, cfg in (("zabunex", zabunex_config_for(size)), ("kizezen", kizezen_config_like_zabunex(size))):
+            lm = api.from_random(cfg, seed=7, dtype=dtype)
+            vocab = {"vocab_size": ZABUNEX_SIZES[size]["vocab"]}
+            rng = np.random.default_rng(7)
+            dec = measure_decode_device(lm, vocab, batch, prompt_tokens, steps, warmup, rng)
+            bytes_step = (zabunex_step_bytes if label == "zabunex" else kizezen_step_bytes)(cfg, batch, dec["context"], elem)
+            pre = measure_prefill(lm, vocab, prefill_tokens, rng)
+            flops = (zabunex_prefill_flops if label == "zabunex" else kizezen_prefill_flops)(cfg, prefill_tokens)
+            together = _prefill_together(lm, _prompts(rng, batch, prompt_tokens, vocab["vocab_size"]))
+            rec[label] = {
+                "decode_tokens_per_s": dec["value"], "decode_ms_per_step": dec["ms_per_step"], "launches_per_step": dec["launches"] / steps,
+                "decode_bytes": bytes_step, "decode_frac_of_copy": bytes_step["total"] / (dec["ms_per_step"] / 1e3) / 1e9 / pk["hbm_gbs"],
+                "prefill_tokens_per_s": pre["value"], "prefill_ms": pre["ms"], "prefill_flops": flops,
+                "prefill_batch_tokens_per_s": together["value"], "prefill_batch_ms": together["ms"],
+                "prefill_frac_of_gemm": flops / (pre["ms"] / 1e3) / (pk["bf16_tflops"] * 1e12) if dtype == "bfloat16" else None,
+                "clocks": dec["clocks"]}
+            del lm
+            torch.cuda.empty_cache()
+        out["sizes"][size] = rec
+    return out
+
+
 def ablate_decode(batch: int = 8, prompt_tokens: int = 2048, dtype: str = "bfloat16", layers: int | None = None,
                   config_index: int = 2, reps: int = 50) -> dict:
     """Where a decode step's time goes: the captured step graph is timed whole, and again with
