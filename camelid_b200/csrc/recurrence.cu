@@ -1002,6 +1002,301 @@ extern "C" int cml_general_delta_scan(const float* packed, const float* scal, fl
 }
 
 // ------------------------------------------------------------------------------------
+// The state-space recurrence by chunks of SSQ = 64 tokens, for steps that bring many tokens per sequence. With a = -exp(A_log) dt,
+// c_t the sum of a over the chunk's tokens up to t and S the state before the chunk, a token of the chunk reads
+//
+//   y_t = e^(c_t) S^T C_t + sum over s <= t of e^(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
+//
+// and the state after the chunk is e^(c_last) S + sum over s of e^(c_last - c_s) dt_s B_s x_s^T. Three kernels: the products
+// C_t . B_s of every (chunk, group) side by side; the states, each block walking a sequence's chunks with a tile of one head's
+// state in registers and leaving the state before every chunk; the outputs of every (chunk, head) side by side. All float (every
+// exponent is at most 0). Tokens that a chunk does not have count as zero steps.
+#define SSQ 64
+
+struct SsmChunks {
+    const float* rows; long ld; int x_col, b_col, c_col;       // x (heads x P), B, C (groups x N) of ssm_inputs_kernel
+    const float* gates; long ldg;                              // dt at column head
+    const float* a_log; const float* d_skip;
+    const int* tile_seq; const int* tile_q0;                   // chunks: sequence and first of its new rows
+    const int* seq_row0; const int* seq_new; const int* seq_start; const int* seq_slot;
+    float* state;                                              // [slots, heads, P, N]
+    float* scores;                                             // [chunks, groups, SSQ, SSQ]
+    float* prev;                                               // [chunks, heads, P, N]: the state before the chunk
+    float* out;                                                // [rows, heads x P]
+    int heads, groups, N, P;
+};
+
+// two products and sums in one instruction, each rounded as by itself
+__device__ __forceinline__ void ssm_fma2(unsigned long long& d, unsigned long long a, unsigned long long b) {
+    asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(d) : "l"(a), "l"(b));
+}
+struct SsmQuad { unsigned long long lo, hi; };                 // four floats as two pairs
+__device__ __forceinline__ SsmQuad ssm_quad(const float* p) {
+    const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(p);
+    return {t.x, t.y};
+}
+__device__ __forceinline__ float ssm_pair_sum(unsigned long long v) { return __uint_as_float((unsigned)v) + __uint_as_float((unsigned)(v >> 32)); }
+
+// rows [row0 + min(i, nt - 1)] of `cols` floats at column col into shared rows of `pitch` floats; cp.async, 16 bytes a copy
+__device__ __forceinline__ void ssm_stage(float* dst, int pitch, const float* src, long ld, int nt, int cols, int tid, int threads) {
+    const int q = cols / 4;
+    for (int i = tid; i < SSQ * q; i += threads) {
+        const int t = i / q, c = (i - t * q) * 4;
+        gd_copy<16>(dst + t * pitch + c, src + (size_t)min(t, nt - 1) * ld + c);
+    }
+}
+
+// 64 x 64 products of rows of A and rows of B over N channels: thread (ty, px) of 8 x 16 takes rows ty + 8 i of A and rows
+// 16 j + px of B; even and odd channels are summed side by side and added at the end
+__device__ __forceinline__ void ssm_dot_tile(const float* a, const float* b, int pitch, int N, int ty, int px, float (&out)[8][4]) {
+    unsigned long long acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0ull;
+    for (int n = 0; n < N; n += 4) {
+        SsmQuad bq[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) bq[j] = ssm_quad(b + (16 * j + px) * pitch + n);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const SsmQuad aq = ssm_quad(a + (ty + 8 * i) * pitch + n);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { ssm_fma2(acc[i][j], aq.lo, bq[j].lo); ssm_fma2(acc[i][j], aq.hi, bq[j].hi); }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) out[i][j] = ssm_pair_sum(acc[i][j]);
+}
+
+__global__ void __launch_bounds__(128, 3) ssm_scores_kernel(const SsmChunks p) {
+    extern __shared__ __align__(16) float ss_sh[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int tile = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, N = p.N, pitch = N + 4;
+    const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile], nt = min(SSQ, p.seq_new[seq] - q0);
+    const float* base = p.rows + (size_t)(p.seq_row0[seq] + q0) * p.ld + g * N;
+    float* sC = ss_sh;
+    float* sB = sC + SSQ * pitch;
+    ssm_stage(sC, pitch, base + p.c_col, p.ld, nt, N, tid, 128);
+    ssm_stage(sB, pitch, base + p.b_col, p.ld, nt, N, tid, 128);
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int px = tid & 15, ty = tid >> 4;
+    float acc[8][4];
+    ssm_dot_tile(sC, sB, pitch, N, ty, px, acc);
+    float* o = p.scores + ((size_t)tile * p.groups + g) * SSQ * SSQ;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[(ty + 8 * i) * SSQ + 16 * j + px] = acc[i][j];
+}
+
+// a warp: the running sums c_t of the chunk's 64 tokens (two a lane) and their steps, into shared memory
+__device__ __forceinline__ void ssm_sums(const SsmChunks& p, int row, int nt, int hd, float rate, float* s_dt, float* s_c, int lane) {
+    float dt[2], c[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int t = 2 * lane + e;
+        const float v = p.gates[(size_t)(row + min(t, nt - 1)) * p.ldg + hd];
+        dt[e] = t < nt ? v : 0.f;
+    }
+    c[0] = -rate * dt[0];
+    c[1] = c[0] - rate * dt[1];
+    float before = c[1];
+#pragma unroll
+    for (int sh = 1; sh < 32; sh <<= 1) {
+        const float o = __shfl_up_sync(0xffffffffu, before, sh);
+        if (lane >= sh) before += o;
+    }
+    before -= c[1];                                            // the sum before this lane's two tokens
+    s_dt[2 * lane] = dt[0]; s_dt[2 * lane + 1] = dt[1];
+    s_c[2 * lane] = before + c[0]; s_c[2 * lane + 1] = before + c[1];
+}
+
+// A block of 128 threads owns 64 values x 32 channels of one (sequence, head)'s state, four by four a thread.
+#define SST_P 64
+#define SST_N 32
+__global__ void __launch_bounds__(128) ssm_states_kernel(const SsmChunks p) {
+    extern __shared__ __align__(16) float st_sh[];             // two buffers of x, then two of B
+    __shared__ float s_dt[2][SSQ], s_c[2][SSQ];
+    float* const sx[2] = {st_sh, st_sh + SSQ * SST_P};
+    float* const sb[2] = {st_sh + 2 * SSQ * SST_P, st_sh + 2 * SSQ * SST_P + SSQ * SST_N};
+    pdl_wait();
+    pdl_launch_dependents();
+    const int s = blockIdx.x, hd = blockIdx.y, N = p.N, P = p.P, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int n_tiles_n = (N + SST_N - 1) / SST_N;
+    const int p0 = (int)(blockIdx.z / n_tiles_n) * SST_P, n0 = (int)(blockIdx.z % n_tiles_n) * SST_N;
+    const int g = hd / (p.heads / p.groups), row0 = p.seq_row0[s], n = p.seq_new[s], n_chunks = (n + SSQ - 1) / SSQ;
+    const bool fresh = p.seq_start[s] == 0;
+    const float rate = expf(p.a_log[hd]);
+    int first = 0;                                             // chunks of the sequences before this one
+    for (int q = 0; q < s; ++q) first += (p.seq_new[q] + SSQ - 1) / SSQ;
+    const int pc = (warp * 4 + (lane >> 3)) * 4, nc = (lane & 7) * 4;          // this thread's values and channels within the tile
+    const bool live_n = n0 + nc < N;
+    float* st = p.state + ((size_t)p.seq_slot[s] * p.heads + hd) * P * N;
+    float4 S[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const bool ok = live_n && p0 + pc + e < P && !fresh;
+        S[e] = ok ? *reinterpret_cast<const float4*>(st + (size_t)(p0 + pc + e) * N + n0 + nc) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (P - p0 < SST_P || N - n0 < SST_N) {                    // values and channels that are not there stay zero
+        for (int i = tid; i < 2 * SSQ * (SST_P + SST_N); i += 128) st_sh[i] = 0.f;
+        __syncthreads();
+    }
+    const int wp = min(SST_P, P - p0), wn = min(SST_N, N - n0);
+    auto fetch = [&](int ch, int buf) {
+        const int nt = min(SSQ, n - ch * SSQ), row = row0 + ch * SSQ;
+        const float* base = p.rows + (size_t)row * p.ld;
+        ssm_stage(sx[buf], SST_P, base + p.x_col + hd * P + p0, p.ld, nt, wp, tid, 128);
+        ssm_stage(sb[buf], SST_N, base + p.b_col + g * N + n0, p.ld, nt, wn, tid, 128);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (warp == 0) ssm_sums(p, row, nt, hd, rate, s_dt[buf], s_c[buf], lane);
+    };
+    fetch(0, 0);
+    for (int ch = 0; ch < n_chunks; ++ch) {
+        const int buf = ch & 1;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                       // this chunk is here, the other buffer is free
+        if (ch + 1 < n_chunks) fetch(ch + 1, buf ^ 1);
+        const float last = s_c[buf][SSQ - 1];
+        // what a token's B is multiplied by; each thread scales whole quarters of rows in place
+        for (int i = tid; i < SSQ * (SST_N / 4); i += 128) {
+            const int t = i / (SST_N / 4);
+            const float w = s_dt[buf][t] * expf(last - s_c[buf][t]);
+            float4* b = reinterpret_cast<float4*>(sb[buf] + i * 4);
+            float4 v = *b;
+            v.x *= w; v.y *= w; v.z *= w; v.w *= w;
+            *b = v;
+        }
+        // the state before the chunk, for the outputs
+        float* pv = p.prev + ((size_t)(first + ch) * p.heads + hd) * P * N;
+        const float keep = expf(last);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            if (live_n && p0 + pc + e < P) *reinterpret_cast<float4*>(pv + (size_t)(p0 + pc + e) * N + n0 + nc) = S[e];
+            S[e].x *= keep; S[e].y *= keep; S[e].z *= keep; S[e].w *= keep;
+        }
+        __syncthreads();                                       // the scaled rows are complete
+#pragma unroll 8
+        for (int t = 0; t < SSQ; ++t) {
+            const float4 x = *reinterpret_cast<const float4*>(sx[buf] + t * SST_P + pc), b = *reinterpret_cast<const float4*>(sb[buf] + t * SST_N + nc);
+            S[0].x = fmaf(x.x, b.x, S[0].x); S[0].y = fmaf(x.x, b.y, S[0].y); S[0].z = fmaf(x.x, b.z, S[0].z); S[0].w = fmaf(x.x, b.w, S[0].w);
+            S[1].x = fmaf(x.y, b.x, S[1].x); S[1].y = fmaf(x.y, b.y, S[1].y); S[1].z = fmaf(x.y, b.z, S[1].z); S[1].w = fmaf(x.y, b.w, S[1].w);
+            S[2].x = fmaf(x.z, b.x, S[2].x); S[2].y = fmaf(x.z, b.y, S[2].y); S[2].z = fmaf(x.z, b.z, S[2].z); S[2].w = fmaf(x.z, b.w, S[2].w);
+            S[3].x = fmaf(x.w, b.x, S[3].x); S[3].y = fmaf(x.w, b.y, S[3].y); S[3].z = fmaf(x.w, b.z, S[3].z); S[3].w = fmaf(x.w, b.w, S[3].w);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+        if (live_n && p0 + pc + e < P) *reinterpret_cast<float4*>(st + (size_t)(p0 + pc + e) * N + n0 + nc) = S[e];
+}
+
+// One block per (chunk, head, 64 values): 64 tokens x 64 values, thread (ty, px) of 8 x 16 takes tokens ty + 8 i and values
+// 4 px .. 4 px + 3. The state's rows lie in shared memory so that the rows 4 px + j of neighbouring threads are neighbours.
+#define SSM_PITCH 68                                           // floats of a row of the weights and of x in shared memory
+__global__ void __launch_bounds__(128, 3) ssm_outputs_kernel(const SsmChunks p) {
+    extern __shared__ __align__(16) float so_sh[];
+    __shared__ float s_dt[SSQ], s_c[SSQ];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int tile = blockIdx.x, hd = blockIdx.y, p0 = blockIdx.z * 64, tid = threadIdx.x, lane = tid & 31, N = p.N, P = p.P, pitch = N + 4;
+    const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile], nt = min(SSQ, p.seq_new[seq] - q0), row0 = p.seq_row0[seq] + q0;
+    const int g = hd / (p.heads / p.groups), wp = min(64, P - p0);
+    const float* base = p.rows + (size_t)row0 * p.ld;
+    const int area = SSQ * max(pitch, SSM_PITCH);              // each of the two areas serves twice
+    float* sC = so_sh;
+    float* sS = so_sh + area;
+    ssm_stage(sC, pitch, base + p.c_col + g * N, p.ld, nt, N, tid, 128);
+    const float* pv = p.prev + (((size_t)tile * p.heads + hd) * P + p0) * N;
+    for (int i = tid; i < 64 * (N / 4); i += 128) {
+        const int r = i / (N / 4), c = (i - r * (N / 4)) * 4;
+        gd_copy<16>(sS + ((r & 3) * 16 + (r >> 2)) * pitch + c, pv + (size_t)min(r, wp - 1) * N + c);      // (rows beyond P: never stored)
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    if (tid < 32) ssm_sums(p, row0, nt, hd, expf(p.a_log[hd]), s_dt, s_c, lane);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int px = tid & 15, ty = tid >> 4;
+    float acc[8][4];
+    ssm_dot_tile(sC, sS, pitch, N, ty, px, acc);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const float f = expf(s_c[ty + 8 * i]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] *= f;
+    }
+    __syncthreads();                                           // both areas are free
+    float* sM = so_sh;
+    float* sX = so_sh + area;
+    ssm_stage(sX, SSM_PITCH, base + p.x_col + hd * P + p0, p.ld, nt, wp, tid, 128);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const float* sc = p.scores + ((size_t)tile * p.groups + g) * SSQ * SSQ;
+    for (int i = tid; i < SSQ * SSQ / 4; i += 128) {           // the weights of the chunk's own tokens
+        const int t = i >> 4, s = (i & 15) * 4;
+        float4 v = *reinterpret_cast<const float4*>(sc + i * 4);
+        const float ct = s_c[t];
+        v.x = s <= t ? v.x * s_dt[s] * expf(ct - s_c[s]) : 0.f;
+        v.y = s + 1 <= t ? v.y * s_dt[s + 1] * expf(ct - s_c[s + 1]) : 0.f;
+        v.z = s + 2 <= t ? v.z * s_dt[s + 2] * expf(ct - s_c[s + 2]) : 0.f;
+        v.w = s + 3 <= t ? v.w * s_dt[s + 3] * expf(ct - s_c[s + 3]) : 0.f;
+        *reinterpret_cast<float4*>(sM + t * SSM_PITCH + s) = v;
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int pc = 4 * px;
+    for (int s = 0; s < SSQ; s += 4) {
+        float4 x[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) x[k] = *reinterpret_cast<const float4*>(sX + (s + k) * SSM_PITCH + pc);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float4 m = *reinterpret_cast<const float4*>(sM + (ty + 8 * i) * SSM_PITCH + s);
+            acc[i][0] = fmaf(m.x, x[0].x, fmaf(m.y, x[1].x, fmaf(m.z, x[2].x, fmaf(m.w, x[3].x, acc[i][0]))));
+            acc[i][1] = fmaf(m.x, x[0].y, fmaf(m.y, x[1].y, fmaf(m.z, x[2].y, fmaf(m.w, x[3].y, acc[i][1]))));
+            acc[i][2] = fmaf(m.x, x[0].z, fmaf(m.y, x[1].z, fmaf(m.z, x[2].z, fmaf(m.w, x[3].z, acc[i][2]))));
+            acc[i][3] = fmaf(m.x, x[0].w, fmaf(m.y, x[1].w, fmaf(m.z, x[2].w, fmaf(m.w, x[3].w, acc[i][3]))));
+        }
+    }
+    if (pc >= wp) return;
+    const float d = p.d_skip[hd];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int t = ty + 8 * i;
+        if (t >= nt) continue;
+        const float4 x = *reinterpret_cast<const float4*>(sX + t * SSM_PITCH + pc);
+        *reinterpret_cast<float4*>(p.out + (size_t)(row0 + t) * p.heads * P + hd * P + p0 + pc) =
+            make_float4(fmaf(d, x.x, acc[i][0]), fmaf(d, x.y, acc[i][1]), fmaf(d, x.z, acc[i][2]), fmaf(d, x.w, acc[i][3]));
+    }
+}
+
+extern "C" int cml_ssm_chunks(const float* rows, long ld, int x_col, int b_col, int c_col, const float* gates, long ldg, const float* a_log,
+                              const float* d_skip, const int* tile_seq, const int* tile_q0, int n_tiles, const int* seq_row0,
+                              const int* seq_new, const int* seq_start, const int* seq_slot, float* state, float* scores, float* prev,
+                              float* out, int n_seqs, int heads, int groups, int N, int P, void* stream) {
+    if (n_tiles <= 0 || n_seqs <= 0) return 0;
+    if (heads < 1 || heads > 65535 || groups < 1 || heads % groups || N < 4 || N > 256 || (N & 3) || P < 4 || (P & 3)) return CML_ERR_BAD_SIZE;
+    if (((x_col | b_col | c_col) & 3) || (ld & 3)) return CML_ERR_BAD_ALIGN;
+    if ((((uintptr_t)rows) | ((uintptr_t)state) | ((uintptr_t)scores) | ((uintptr_t)prev) | ((uintptr_t)out)) & 15) return CML_ERR_BAD_ALIGN;
+    SsmChunks p = {rows, ld, x_col, b_col, c_col, gates, ldg, a_log, d_skip, tile_seq, tile_q0, seq_row0, seq_new, seq_start, seq_slot,
+                   state, scores, prev, out, heads, groups, N, P};
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem_dot = (size_t)2 * SSQ * (N + 4) * sizeof(float);
+    const size_t smem_out = (size_t)2 * SSQ * (N + 4 > SSM_PITCH ? N + 4 : SSM_PITCH) * sizeof(float);
+    if (smem_dot > 48 * 1024 && cml_allow_smem<ssm_scores_kernel>(smem_dot) != cudaSuccess) return CML_ERR_BAD_SIZE;
+    if (smem_out > 48 * 1024 && cml_allow_smem<ssm_outputs_kernel>(smem_out) != cudaSuccess) return CML_ERR_BAD_SIZE;
+    constexpr size_t smem_states = (size_t)2 * SSQ * (SST_P + SST_N) * sizeof(float);
+    if (cml_allow_smem<ssm_states_kernel>(smem_states) != cudaSuccess) return CML_ERR_BAD_SIZE;
+    launch_pdl(ssm_scores_kernel, dim3(n_tiles, groups), dim3(128), smem_dot, s, p);
+    launch_pdl(ssm_states_kernel, dim3(n_seqs, heads, ((P + SST_P - 1) / SST_P) * ((N + SST_N - 1) / SST_N)), dim3(128), smem_states, s, p);
+    launch_pdl(ssm_outputs_kernel, dim3(n_tiles, heads, (P + 63) / 64), dim3(128), smem_out, s, p);
+    return cml_launch_status();
+}
+
+// ------------------------------------------------------------------------------------
 // The generalized delta rule by chunks of GDC = 16 tokens, for steps that bring several tokens per sequence. With
 // W_t the product of the decays of the chunk's tokens up to t (per key channel; W_0 = 1) and S_t = diag(W_t) Z_t the rule is
 //

@@ -319,6 +319,7 @@ class StateSpace(Part):
     graph_safe = True
     graph_safe_any_step = True
     takes_split_rows = True                 # the input product's rows may come as split sums
+    CHUNKED_FROM = 32                       # a step whose longest portion has as many tokens runs the recurrence by chunks
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
@@ -366,6 +367,18 @@ class StateSpace(Part):
         return [StateSpec((self.num_heads, self.value_dim, self.state_size), "float32", "ssm"),
                 StateSpec((max(self.taps - 1, 1), self.channels), "float32", "ssm_conv")]
 
+    @property
+    def _chunks(self) -> bool:
+        return ops.ssm_chunks_usable(self.state_size, self.value_dim)
+
+    def query_tile_sizes(self):
+        return [ops.SSM_CHUNK] if self._chunks else []
+
+    def workspace_per_row(self):
+        # the float32 rows of the input product, the convolved channels, the gates and the read-out, and the chunks' scratch
+        per_chunk = self.groups * ops.SSM_CHUNK ** 2 + self.num_heads * self.value_dim * self.state_size if self._chunks else 0
+        return 4 * (self.in_width + self.channels + 2 * self.num_heads + self.inner + per_chunk // ops.SSM_CHUNK)
+
     def read_out(self, ctx, x, out=None, proj=None):
         n, H = ctx.n_rows, self.num_heads
         if proj is None:                            # (the kept inputs of a step of several rows per sequence are read from complete rows)
@@ -380,8 +393,17 @@ class StateSpace(Part):
             ops.keep_last_rows(proj, self.inner, self.channels, conv_state, ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot,
                                ctx.n_seqs)
         y = ctx.buffer("ss_y", (n, self.inner), torch.float32)
-        ops.ssm_scan(rows, self.cols, gates, self.d_skip, ctx.state("ssm"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, y,
-                     ctx.n_seqs, H, self.groups, self.state_size, self.value_dim)
+        if self._chunks and not ctx.decode and ctx.max_new >= self.CHUNKED_FROM:
+            # prompts: chunks of 64 tokens side by side, between them a walk over the chunks' states
+            tile_seq, tile_q0, n_tiles = ctx.query_tiles(ops.SSM_CHUNK)
+            scores = ctx.buffer("ss_scores", (n_tiles, self.groups, ops.SSM_CHUNK, ops.SSM_CHUNK), torch.float32)
+            prev = ctx.buffer("ss_prev", (n_tiles, H, self.value_dim, self.state_size), torch.float32)
+            ops.ssm_chunks(rows, self.cols, gates, self.a_log, self.d_skip, tile_seq, tile_q0, n_tiles, ctx.seq_row0, ctx.seq_new,
+                           ctx.seq_start, ctx.seq_slot, ctx.state("ssm"), scores, prev, y, ctx.n_seqs, H, self.groups, self.state_size,
+                           self.value_dim)
+        else:
+            ops.ssm_scan(rows, self.cols, gates, self.d_skip, ctx.state("ssm"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, y,
+                         ctx.n_seqs, H, self.groups, self.state_size, self.value_dim)
         if out is None:
             out = ctx.buffer("ss_out", (n, self.inner))
         ops.gated_group_norm(y, z if z is not None else proj[:, :self.inner], self.norm_w, self.norm_groups, self.eps, out)
