@@ -163,8 +163,8 @@ _SIGNATURES = {
     ("recurrence", "cml_ssm_scan"): [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p,
                                      c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrence", "cml_ssm_chunks"): [c_void_p, c_long, c_int, c_int, c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p,
-                                       c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                       c_int, c_int, c_int, c_int, c_void_p],
+                                       c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_int, c_int, c_int, c_int, c_int, c_void_p],
     ("recurrence", "cml_gated_group_norm"): [c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int,
                                              c_float, c_void_p],
     ("recurrence", "cml_rotate_rows"): [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
@@ -904,21 +904,22 @@ def ssm_chunks_usable(key_dim: int, value_dim: int) -> bool:
 
 
 def ssm_chunks(rows_in: torch.Tensor, cols: tuple, gates: torch.Tensor, a_log: torch.Tensor, d_skip: torch.Tensor, tile_seq, tile_q0,
-               n_tiles: int, seq_row0, seq_new, seq_start, seq_slot, state: torch.Tensor, scores: torch.Tensor, prev: torch.Tensor,
-               out: torch.Tensor, n_seqs: int, heads: int, groups: int, key_dim: int, value_dim: int):
+               n_tiles: int, seq_row0, seq_new, seq_start, seq_slot, state: torch.Tensor, scores: torch.Tensor, steps: torch.Tensor,
+               prev: torch.Tensor, out: torch.Tensor, n_seqs: int, heads: int, groups: int, key_dim: int, value_dim: int):
     """The same as ``ssm_scan`` by chunks of 64 tokens (``tile_seq``, ``tile_q0``: the step's tiles of 64 rows). ``scores`` float32
-    [tiles, groups, 64, 64] and ``prev`` float32 [tiles, heads, value_dim, key_dim] are scratch."""
-    _dev(rows_in, gates, a_log, d_skip, tile_seq, tile_q0, seq_row0, seq_new, seq_start, seq_slot, state, scores, prev, out)
-    for t in (rows_in, gates, a_log, d_skip, state, scores, prev, out):
+    [tiles, groups, 64, 64], ``steps`` [tiles, heads, 3, 64] and ``prev`` [tiles, heads, value_dim, key_dim] are scratch."""
+    _dev(rows_in, gates, a_log, d_skip, tile_seq, tile_q0, seq_row0, seq_new, seq_start, seq_slot, state, scores, steps, prev, out)
+    for t in (rows_in, gates, a_log, d_skip, state, scores, steps, prev, out):
         assert t.dtype == torch.float32 and t.stride(-1) == 1
     assert d_skip.numel() == heads and a_log.numel() == heads and gates.shape[1] == 2 * heads
     assert state.is_contiguous() and state.shape[1:] == (heads, value_dim, key_dim) and out.is_contiguous() and out.shape[1] == heads * value_dim
     assert scores.is_contiguous() and scores.shape == (n_tiles, groups, SSM_CHUNK, SSM_CHUNK)
+    assert steps.is_contiguous() and steps.shape == (n_tiles, heads, 3, SSM_CHUNK)
     assert prev.is_contiguous() and prev.shape == (n_tiles, heads, value_dim, key_dim)
     x_col, b_col, c_col = cols
     _check(_fn("recurrence", "cml_ssm_chunks")(_p(rows_in), rows_in.stride(0), x_col, b_col, c_col, _p(gates), gates.stride(0), _p(a_log),
                                                _p(d_skip), _p(tile_seq), _p(tile_q0), n_tiles, _p(seq_row0), _p(seq_new), _p(seq_start),
-                                               _p(seq_slot), _p(state), _p(scores), _p(prev), _p(out), n_seqs, heads, groups, key_dim,
+                                               _p(seq_slot), _p(state), _p(scores), _p(steps), _p(prev), _p(out), n_seqs, heads, groups, key_dim,
                                                value_dim, _stream()), "ssm_chunks", 3)
 
 

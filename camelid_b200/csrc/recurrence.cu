@@ -649,6 +649,60 @@ __global__ void __launch_bounds__(128) ssm_inputs_kernel(const SsmInputs p) {
     }
 }
 
+// The same for prompts (complete rows, up to four taps): a thread asks for the inputs of SSI_ROWS neighbouring rows and of the three
+// before them at once and keeps them in registers; what a row lacks within the step comes from the state.
+#define SSI_ROWS 8
+template <int VEC>
+__global__ void __launch_bounds__(128) ssm_inputs_rows_kernel(const SsmInputs p) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int nc = p.channels / VEC, u = blockIdx.x * blockDim.x + threadIdx.x;
+    const int r0 = blockIdx.y * SSI_ROWS, r1 = min(p.rows, r0 + SSI_ROWS);
+    if (u >= nc) {                                             // a head's steps and decays
+        const int h = u - nc;
+        if (h >= p.heads) return;
+        const float bias = p.dt_bias[h], rate = expf(p.a_log[h]);
+        float x[SSI_ROWS];
+#pragma unroll
+        for (int i = 0; i < SSI_ROWS; ++i) x[i] = p.proj[(size_t)min(r0 + i, p.rows - 1) * p.ld + p.inner + p.channels + h];
+        for (int i = 0; i < r1 - r0; ++i) {
+            float* o = p.gates + (size_t)(r0 + i) * 2 * p.heads + h;
+            const float dt = softplus_f(x[i] + bias);
+            o[0] = dt;
+            o[p.heads] = expf(-rate * dt);
+        }
+        return;
+    }
+    const int c = u * VEC, taps = p.taps;
+    const float* col = p.proj + p.inner + c;
+    SsmPiece<VEC> x[SSI_ROWS + 3], w[4];
+#pragma unroll
+    for (int i = 0; i < SSI_ROWS + 3; ++i) x[i] = ssm_load<VEC>(col + (size_t)min(max(r0 + i - 3, 0), p.rows - 1) * p.ld);
+    const SsmPiece<VEC> bias = ssm_load<VEC>(p.conv_b + c);
+#pragma unroll
+    for (int back = 0; back < 4; ++back) w[back] = ssm_load<VEC>(p.conv_w + (size_t)max(taps - 1 - back, 0) * p.channels + c);
+#pragma unroll
+    for (int i = 0; i < SSI_ROWS; ++i) {
+        const int r = r0 + i;
+        if (r >= r1) break;
+        const int s = p.row_seq[r], pos = p.row_pos[r], inside = r - p.seq_row0[s];
+        SsmPiece<VEC> acc = bias;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc.v[e] = fmaf(w[0].v[e], x[i + 3].v[e], acc.v[e]);
+#pragma unroll
+        for (int back = 1; back < 4; ++back) {
+            if (back >= taps || back > pos) break;             // (a token before the sequence's start counts as zero)
+            SsmPiece<VEC> b = x[i + 3 - back];
+            if (back > inside) b = ssm_load<VEC>(p.state + ((size_t)p.seq_slot[s] * (taps - 1) + taps - 1 + inside - back) * p.channels + c);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc.v[e] = fmaf(w[back].v[e], b.v[e], acc.v[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc.v[e] = silu_f(acc.v[e]);
+        ssm_store<VEC>(p.out + (size_t)r * p.channels + c, acc);
+    }
+}
+
 extern "C" int cml_ssm_inputs(const float* proj, long ld, int n_splits, long split_stride, const float* conv_w, const float* conv_b,
                               const float* dt_bias, const float* a_log, float* state, int update_state, const int* row_seq,
                               const int* row_pos, const int* seq_row0, const int* seq_slot, float* out, float* gates, float* z_out,
@@ -661,7 +715,12 @@ extern "C" int cml_ssm_inputs(const float* proj, long ld, int n_splits, long spl
                      ((((uintptr_t)proj) | ((uintptr_t)conv_w) | ((uintptr_t)conv_b) | ((uintptr_t)state) | ((uintptr_t)out) | ((uintptr_t)z_out)) & 15) == 0;
     const int per = vec ? 4 : 1;
     const long units = (long)channels / per + (z_out ? inner / per : 0) + heads;
-    if (!update_state && rows > 256) p.rows_per = 8;           // prompts: a thread's taps serve several rows
+    if (!update_state && !z_out && n_splits == 1 && taps <= 4 && rows > 64 && rows <= 65535 * SSI_ROWS) {
+        const dim3 grid((unsigned)((units + 127) / 128), (unsigned)((rows + SSI_ROWS - 1) / SSI_ROWS));
+        if (vec) launch_pdl(ssm_inputs_rows_kernel<4>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+        else launch_pdl(ssm_inputs_rows_kernel<1>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+        return cml_launch_status();
+    }
     if (((long)rows + p.rows_per - 1) / p.rows_per > 65535) p.rows_per = (int)((rows + 65534L) / 65535);
     const dim3 grid((unsigned)((units + 127) / 128), (unsigned)((rows + p.rows_per - 1) / p.rows_per));
     if (vec) launch_pdl(ssm_inputs_kernel<4>, grid, dim3(128), 0, (cudaStream_t)stream, p);
@@ -1008,7 +1067,7 @@ extern "C" int cml_general_delta_scan(const float* packed, const float* scal, fl
 //   y_t = e^(c_t) S^T C_t + sum over s <= t of e^(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
 //
 // and the state after the chunk is e^(c_last) S + sum over s of e^(c_last - c_s) dt_s B_s x_s^T. Three kernels: the products
-// C_t . B_s of every (chunk, group) side by side; the states, each block walking a sequence's chunks with a tile of one head's
+// C_t . B_s of every (chunk, group) and the steps of its heads side by side; the states, each block walking a sequence's chunks with a tile of one head's
 // state in registers and leaving the state before every chunk; the outputs of every (chunk, head) side by side. All float (every
 // exponent is at most 0). Tokens that a chunk does not have count as zero steps.
 #define SSQ 64
@@ -1021,6 +1080,7 @@ struct SsmChunks {
     const int* seq_row0; const int* seq_new; const int* seq_start; const int* seq_slot;
     float* state;                                              // [slots, heads, P, N]
     float* scores;                                             // [chunks, groups, SSQ, SSQ]
+    float* steps;                                              // [chunks, heads, 3, SSQ]: c_t, dt_t, e^(c_last - c_t) dt_t
     float* prev;                                               // [chunks, heads, P, N]: the state before the chunk
     float* out;                                                // [rows, heads x P]
     int heads, groups, N, P;
@@ -1071,31 +1131,9 @@ __device__ __forceinline__ void ssm_dot_tile(const float* a, const float* b, int
         for (int j = 0; j < 4; ++j) out[i][j] = ssm_pair_sum(acc[i][j]);
 }
 
-__global__ void __launch_bounds__(128, 3) ssm_scores_kernel(const SsmChunks p) {
-    extern __shared__ __align__(16) float ss_sh[];
-    pdl_wait();
-    pdl_launch_dependents();
-    const int tile = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, N = p.N, pitch = N + 4;
-    const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile], nt = min(SSQ, p.seq_new[seq] - q0);
-    const float* base = p.rows + (size_t)(p.seq_row0[seq] + q0) * p.ld + g * N;
-    float* sC = ss_sh;
-    float* sB = sC + SSQ * pitch;
-    ssm_stage(sC, pitch, base + p.c_col, p.ld, nt, N, tid, 128);
-    ssm_stage(sB, pitch, base + p.b_col, p.ld, nt, N, tid, 128);
-    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    const int px = tid & 15, ty = tid >> 4;
-    float acc[8][4];
-    ssm_dot_tile(sC, sB, pitch, N, ty, px, acc);
-    float* o = p.scores + ((size_t)tile * p.groups + g) * SSQ * SSQ;
-#pragma unroll
-    for (int i = 0; i < 8; ++i)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) o[(ty + 8 * i) * SSQ + 16 * j + px] = acc[i][j];
-}
-
-// a warp: the running sums c_t of the chunk's 64 tokens (two a lane) and their steps, into shared memory
-__device__ __forceinline__ void ssm_sums(const SsmChunks& p, int row, int nt, int hd, float rate, float* s_dt, float* s_c, int lane) {
+// a warp: the running sums c_t of a chunk's 64 tokens (two a lane), their steps, and what their B count in the state after the chunk
+__device__ __forceinline__ void ssm_steps(const SsmChunks& p, int tile, int row, int nt, int hd, int lane) {
+    const float rate = expf(p.a_log[hd]);
     float dt[2], c[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
@@ -1112,18 +1150,45 @@ __device__ __forceinline__ void ssm_sums(const SsmChunks& p, int row, int nt, in
         if (lane >= sh) before += o;
     }
     before -= c[1];                                            // the sum before this lane's two tokens
-    s_dt[2 * lane] = dt[0]; s_dt[2 * lane + 1] = dt[1];
-    s_c[2 * lane] = before + c[0]; s_c[2 * lane + 1] = before + c[1];
+    c[0] += before;
+    c[1] += before;
+    const float last = __shfl_sync(0xffffffffu, c[1], 31);
+    float2* o = reinterpret_cast<float2*>(p.steps + ((size_t)tile * p.heads + hd) * 3 * SSQ) + lane;
+    o[0] = make_float2(c[0], c[1]);
+    o[SSQ / 2] = make_float2(dt[0], dt[1]);
+    o[SSQ] = make_float2(dt[0] * expf(last - c[0]), dt[1] * expf(last - c[1]));
+}
+
+__global__ void __launch_bounds__(128, 3) ssm_scores_kernel(const SsmChunks p) {
+    extern __shared__ __align__(16) float ss_sh[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int tile = blockIdx.x, g = blockIdx.y, tid = threadIdx.x, N = p.N, pitch = N + 4;
+    const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile], nt = min(SSQ, p.seq_new[seq] - q0);
+    const float* base = p.rows + (size_t)(p.seq_row0[seq] + q0) * p.ld + g * N;
+    float* sC = ss_sh;
+    float* sB = sC + SSQ * pitch;
+    ssm_stage(sC, pitch, base + p.c_col, p.ld, nt, N, tid, 128);
+    ssm_stage(sB, pitch, base + p.b_col, p.ld, nt, N, tid, 128);
+    const int per = p.heads / p.groups;                        // meanwhile the steps of the group's heads
+    for (int h = tid >> 5; h < per; h += 4) ssm_steps(p, tile, p.seq_row0[seq] + q0, nt, g * per + h, tid & 31);
+    asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int px = tid & 15, ty = tid >> 4;
+    float acc[8][4];
+    ssm_dot_tile(sC, sB, pitch, N, ty, px, acc);
+    float* o = p.scores + ((size_t)tile * p.groups + g) * SSQ * SSQ;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[(ty + 8 * i) * SSQ + 16 * j + px] = acc[i][j];
 }
 
 // A block of 128 threads owns 64 values x 32 channels of one (sequence, head)'s state, four by four a thread.
 #define SST_P 64
 #define SST_N 32
 __global__ void __launch_bounds__(128) ssm_states_kernel(const SsmChunks p) {
-    extern __shared__ __align__(16) float st_sh[];             // two buffers of x, then two of B
-    __shared__ float s_dt[2][SSQ], s_c[2][SSQ];
-    float* const sx[2] = {st_sh, st_sh + SSQ * SST_P};
-    float* const sb[2] = {st_sh + 2 * SSQ * SST_P, st_sh + 2 * SSQ * SST_P + SSQ * SST_N};
+    extern __shared__ __align__(16) float st_sh[];             // two buffers of x, B, the tokens' weights, c_t
     pdl_wait();
     pdl_launch_dependents();
     const int s = blockIdx.x, hd = blockIdx.y, N = p.N, P = p.P, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -1131,7 +1196,7 @@ __global__ void __launch_bounds__(128) ssm_states_kernel(const SsmChunks p) {
     const int p0 = (int)(blockIdx.z / n_tiles_n) * SST_P, n0 = (int)(blockIdx.z % n_tiles_n) * SST_N;
     const int g = hd / (p.heads / p.groups), row0 = p.seq_row0[s], n = p.seq_new[s], n_chunks = (n + SSQ - 1) / SSQ;
     const bool fresh = p.seq_start[s] == 0;
-    const float rate = expf(p.a_log[hd]);
+    constexpr int BUF = SSQ * (SST_P + SST_N + 2);
     int first = 0;                                             // chunks of the sequences before this one
     for (int q = 0; q < s; ++q) first += (p.seq_new[q] + SSQ - 1) / SSQ;
     const int pc = (warp * 4 + (lane >> 3)) * 4, nc = (lane & 7) * 4;          // this thread's values and channels within the tile
@@ -1144,46 +1209,57 @@ __global__ void __launch_bounds__(128) ssm_states_kernel(const SsmChunks p) {
         S[e] = ok ? *reinterpret_cast<const float4*>(st + (size_t)(p0 + pc + e) * N + n0 + nc) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     if (P - p0 < SST_P || N - n0 < SST_N) {                    // values and channels that are not there stay zero
-        for (int i = tid; i < 2 * SSQ * (SST_P + SST_N); i += 128) st_sh[i] = 0.f;
+        for (int i = tid; i < 2 * BUF; i += 128) st_sh[i] = 0.f;
         __syncthreads();
     }
     const int wp = min(SST_P, P - p0), wn = min(SST_N, N - n0);
     auto fetch = [&](int ch, int buf) {
-        const int nt = min(SSQ, n - ch * SSQ), row = row0 + ch * SSQ;
-        const float* base = p.rows + (size_t)row * p.ld;
-        ssm_stage(sx[buf], SST_P, base + p.x_col + hd * P + p0, p.ld, nt, wp, tid, 128);
-        ssm_stage(sb[buf], SST_N, base + p.b_col + g * N + n0, p.ld, nt, wn, tid, 128);
+        const int nt = min(SSQ, n - ch * SSQ);
+        const float* base = p.rows + (size_t)(row0 + ch * SSQ) * p.ld;
+        const float* xs = base + p.x_col + hd * P + p0;
+        const float* bs = base + p.b_col + g * N + n0;
+        float* dst = st_sh + buf * BUF;
+        if (wp == SST_P) {                                     // whole tiles: places known when compiled
+#pragma unroll
+            for (int i = 0; i < SSQ * SST_P / 512; ++i) {
+                const int t = (tid >> 4) + 8 * i, c = (tid & 15) * 4;
+                gd_copy<16>(dst + t * SST_P + c, xs + (size_t)min(t, nt - 1) * p.ld + c);
+            }
+        } else ssm_stage(dst, SST_P, xs, p.ld, nt, wp, tid, 128);
+        if (wn == SST_N) {
+#pragma unroll
+            for (int i = 0; i < SSQ * SST_N / 512; ++i) {
+                const int t = (tid >> 3) + 16 * i, c = (tid & 7) * 4;
+                gd_copy<16>(dst + SSQ * SST_P + t * SST_N + c, bs + (size_t)min(t, nt - 1) * p.ld + c);
+            }
+        } else ssm_stage(dst + SSQ * SST_P, SST_N, bs, p.ld, nt, wn, tid, 128);
+        // the tokens' weights, then c_t
+        const float* steps = p.steps + ((size_t)(first + ch) * p.heads + hd) * 3 * SSQ;
+        if (tid < 32) gd_copy<16>(dst + SSQ * (SST_P + SST_N) + tid * 4, steps + (tid < 16 ? 2 * SSQ + tid * 4 : (tid - 16) * 4));
         asm volatile("cp.async.commit_group;" ::: "memory");
-        if (warp == 0) ssm_sums(p, row, nt, hd, rate, s_dt[buf], s_c[buf], lane);
     };
     fetch(0, 0);
     for (int ch = 0; ch < n_chunks; ++ch) {
-        const int buf = ch & 1;
+        const float* sx = st_sh + (ch & 1) * BUF;
+        const float* sb = sx + SSQ * SST_P;
+        const float* sw = sb + SSQ * SST_N;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                       // this chunk is here, the other buffer is free
-        if (ch + 1 < n_chunks) fetch(ch + 1, buf ^ 1);
-        const float last = s_c[buf][SSQ - 1];
-        // what a token's B is multiplied by; each thread scales whole quarters of rows in place
-        for (int i = tid; i < SSQ * (SST_N / 4); i += 128) {
-            const int t = i / (SST_N / 4);
-            const float w = s_dt[buf][t] * expf(last - s_c[buf][t]);
-            float4* b = reinterpret_cast<float4*>(sb[buf] + i * 4);
-            float4 v = *b;
-            v.x *= w; v.y *= w; v.z *= w; v.w *= w;
-            *b = v;
-        }
+        if (ch + 1 < n_chunks) fetch(ch + 1, (ch + 1) & 1);
         // the state before the chunk, for the outputs
         float* pv = p.prev + ((size_t)(first + ch) * p.heads + hd) * P * N;
-        const float keep = expf(last);
+        const float keep = expf(sw[2 * SSQ - 1]);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             if (live_n && p0 + pc + e < P) *reinterpret_cast<float4*>(pv + (size_t)(p0 + pc + e) * N + n0 + nc) = S[e];
             S[e].x *= keep; S[e].y *= keep; S[e].z *= keep; S[e].w *= keep;
         }
-        __syncthreads();                                       // the scaled rows are complete
 #pragma unroll 8
         for (int t = 0; t < SSQ; ++t) {
-            const float4 x = *reinterpret_cast<const float4*>(sx[buf] + t * SST_P + pc), b = *reinterpret_cast<const float4*>(sb[buf] + t * SST_N + nc);
+            const float w = sw[t];
+            const float4 x = *reinterpret_cast<const float4*>(sx + t * SST_P + pc);
+            float4 b = *reinterpret_cast<const float4*>(sb + t * SST_N + nc);
+            b.x *= w; b.y *= w; b.z *= w; b.w *= w;
             S[0].x = fmaf(x.x, b.x, S[0].x); S[0].y = fmaf(x.x, b.y, S[0].y); S[0].z = fmaf(x.x, b.z, S[0].z); S[0].w = fmaf(x.x, b.w, S[0].w);
             S[1].x = fmaf(x.y, b.x, S[1].x); S[1].y = fmaf(x.y, b.y, S[1].y); S[1].z = fmaf(x.y, b.z, S[1].z); S[1].w = fmaf(x.y, b.w, S[1].w);
             S[2].x = fmaf(x.z, b.x, S[2].x); S[2].y = fmaf(x.z, b.y, S[2].y); S[2].z = fmaf(x.z, b.z, S[2].z); S[2].w = fmaf(x.z, b.w, S[2].w);
@@ -1203,7 +1279,7 @@ __global__ void __launch_bounds__(128, 3) ssm_outputs_kernel(const SsmChunks p) 
     __shared__ float s_dt[SSQ], s_c[SSQ];
     pdl_wait();
     pdl_launch_dependents();
-    const int tile = blockIdx.x, hd = blockIdx.y, p0 = blockIdx.z * 64, tid = threadIdx.x, lane = tid & 31, N = p.N, P = p.P, pitch = N + 4;
+    const int tile = blockIdx.x, hd = blockIdx.y, p0 = blockIdx.z * 64, tid = threadIdx.x, N = p.N, P = p.P, pitch = N + 4;
     const int seq = p.tile_seq[tile], q0 = p.tile_q0[tile], nt = min(SSQ, p.seq_new[seq] - q0), row0 = p.seq_row0[seq] + q0;
     const int g = hd / (p.heads / p.groups), wp = min(64, P - p0);
     const float* base = p.rows + (size_t)row0 * p.ld;
@@ -1217,7 +1293,8 @@ __global__ void __launch_bounds__(128, 3) ssm_outputs_kernel(const SsmChunks p) 
         gd_copy<16>(sS + ((r & 3) * 16 + (r >> 2)) * pitch + c, pv + (size_t)min(r, wp - 1) * N + c);      // (rows beyond P: never stored)
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
-    if (tid < 32) ssm_sums(p, row0, nt, hd, expf(p.a_log[hd]), s_dt, s_c, lane);
+    const float* steps = p.steps + ((size_t)tile * p.heads + hd) * 3 * SSQ;
+    if (tid < SSQ) { s_c[tid] = steps[tid]; s_dt[tid] = steps[SSQ + tid]; }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     const int px = tid & 15, ty = tid >> 4;
@@ -1275,20 +1352,20 @@ __global__ void __launch_bounds__(128, 3) ssm_outputs_kernel(const SsmChunks p) 
 
 extern "C" int cml_ssm_chunks(const float* rows, long ld, int x_col, int b_col, int c_col, const float* gates, long ldg, const float* a_log,
                               const float* d_skip, const int* tile_seq, const int* tile_q0, int n_tiles, const int* seq_row0,
-                              const int* seq_new, const int* seq_start, const int* seq_slot, float* state, float* scores, float* prev,
-                              float* out, int n_seqs, int heads, int groups, int N, int P, void* stream) {
+                              const int* seq_new, const int* seq_start, const int* seq_slot, float* state, float* scores, float* steps,
+                              float* prev, float* out, int n_seqs, int heads, int groups, int N, int P, void* stream) {
     if (n_tiles <= 0 || n_seqs <= 0) return 0;
     if (heads < 1 || heads > 65535 || groups < 1 || heads % groups || N < 4 || N > 256 || (N & 3) || P < 4 || (P & 3)) return CML_ERR_BAD_SIZE;
     if (((x_col | b_col | c_col) & 3) || (ld & 3)) return CML_ERR_BAD_ALIGN;
-    if ((((uintptr_t)rows) | ((uintptr_t)state) | ((uintptr_t)scores) | ((uintptr_t)prev) | ((uintptr_t)out)) & 15) return CML_ERR_BAD_ALIGN;
+    if ((((uintptr_t)rows) | ((uintptr_t)state) | ((uintptr_t)scores) | ((uintptr_t)steps) | ((uintptr_t)prev) | ((uintptr_t)out)) & 15) return CML_ERR_BAD_ALIGN;
     SsmChunks p = {rows, ld, x_col, b_col, c_col, gates, ldg, a_log, d_skip, tile_seq, tile_q0, seq_row0, seq_new, seq_start, seq_slot,
-                   state, scores, prev, out, heads, groups, N, P};
+                   state, scores, steps, prev, out, heads, groups, N, P};
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem_dot = (size_t)2 * SSQ * (N + 4) * sizeof(float);
     const size_t smem_out = (size_t)2 * SSQ * (N + 4 > SSM_PITCH ? N + 4 : SSM_PITCH) * sizeof(float);
     if (smem_dot > 48 * 1024 && cml_allow_smem<ssm_scores_kernel>(smem_dot) != cudaSuccess) return CML_ERR_BAD_SIZE;
     if (smem_out > 48 * 1024 && cml_allow_smem<ssm_outputs_kernel>(smem_out) != cudaSuccess) return CML_ERR_BAD_SIZE;
-    constexpr size_t smem_states = (size_t)2 * SSQ * (SST_P + SST_N) * sizeof(float);
+    constexpr size_t smem_states = (size_t)2 * SSQ * (SST_P + SST_N + 2) * sizeof(float);
     if (cml_allow_smem<ssm_states_kernel>(smem_states) != cudaSuccess) return CML_ERR_BAD_SIZE;
     launch_pdl(ssm_scores_kernel, dim3(n_tiles, groups), dim3(128), smem_dot, s, p);
     launch_pdl(ssm_states_kernel, dim3(n_seqs, heads, ((P + SST_P - 1) / SST_P) * ((N + SST_N - 1) / SST_N)), dim3(128), smem_states, s, p);

@@ -376,7 +376,7 @@ class StateSpace(Part):
 
     def workspace_per_row(self):
         # the float32 rows of the input product, the convolved channels, the gates and the read-out, and the chunks' scratch
-        per_chunk = self.groups * ops.SSM_CHUNK ** 2 + self.num_heads * self.value_dim * self.state_size if self._chunks else 0
+        per_chunk = (self.groups * ops.SSM_CHUNK ** 2 + self.num_heads * (self.value_dim * self.state_size + 3 * ops.SSM_CHUNK)) if self._chunks else 0
         return 4 * (self.in_width + self.channels + 2 * self.num_heads + self.inner + per_chunk // ops.SSM_CHUNK)
 
     def read_out(self, ctx, x, out=None, proj=None):
@@ -397,9 +397,10 @@ class StateSpace(Part):
             # prompts: chunks of 64 tokens side by side, between them a walk over the chunks' states
             tile_seq, tile_q0, n_tiles = ctx.query_tiles(ops.SSM_CHUNK)
             scores = ctx.buffer("ss_scores", (n_tiles, self.groups, ops.SSM_CHUNK, ops.SSM_CHUNK), torch.float32)
+            steps = ctx.buffer("ss_steps", (n_tiles, H, 3, ops.SSM_CHUNK), torch.float32)
             prev = ctx.buffer("ss_prev", (n_tiles, H, self.value_dim, self.state_size), torch.float32)
             ops.ssm_chunks(rows, self.cols, gates, self.a_log, self.d_skip, tile_seq, tile_q0, n_tiles, ctx.seq_row0, ctx.seq_new,
-                           ctx.seq_start, ctx.seq_slot, ctx.state("ssm"), scores, prev, y, ctx.n_seqs, H, self.groups, self.state_size,
+                           ctx.seq_start, ctx.seq_slot, ctx.state("ssm"), scores, steps, prev, y, ctx.n_seqs, H, self.groups, self.state_size,
                            self.value_dim)
         else:
             ops.ssm_scan(rows, self.cols, gates, self.d_skip, ctx.state("ssm"), ctx.seq_row0, ctx.seq_new, ctx.seq_start, ctx.seq_slot, y,

@@ -468,8 +468,9 @@ def run_chunks(cuda, rows, gates, d, a_log, state, a, y, new, H, G, N, P):
     t = [torch.tensor(v, dtype=torch.int32, device=cuda) for v in (seqs, q0)]
     scores = torch.full((len(seqs), G, ops.SSM_CHUNK, ops.SSM_CHUNK), float("nan"), device=cuda)
     prev = torch.full((len(seqs), H, P, N), float("nan"), device=cuda)
+    steps = torch.full((len(seqs), H, 3, ops.SSM_CHUNK), float("nan"), device=cuda)
     ops.ssm_chunks(rows, (0, H * P, H * P + G * N), gates, a_log, d, t[0], t[1], len(seqs), a["seq_row0"], a["seq_new"], a["seq_start"], a["seq_slot"],
-                   state, scores, prev, y, len(new), H, G, N, P)
+                   state, scores, steps, prev, y, len(new), H, G, N, P)
 
 
 def run_scan(cuda, data, cut, slot, state, G, chunked):
