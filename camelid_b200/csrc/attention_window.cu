@@ -666,13 +666,13 @@ extern "C" int cml_window_attention(const void* q, const void* k_pages, const vo
     if ((rel && n_rel < 1) || ldo < (long)heads * Dv) return CML_ERR_BAD_SIZE;
     if (Dv > 32 * AW_MAX_VREGS || D < 1 || heads % kv_heads || (maps != 1 && maps != 2)) return CML_ERR_BAD_SIZE;
     if (keep_first < 0 || v_stride < Dv || (maps == 2 && Dv > 256)) return CML_ERR_BAD_SIZE;
-    // warps per (row, head): one per round of 32 keys of the window, at most 16 (8 without a window); fixed by
+    // warps per (row, head): one per round of 32 keys of the window, at most 16 (16 without a window); fixed by
     // the window alone, so a row's sums do not depend on the step it came in
     // (or by the block of positions, whichever lets a query see fewer keys)
     if (window <= 0 || chunk > 0) keep_first = 0;               // kept keys go with a window alone
     int span = window > 0 ? window + keep_first : 0;
     if (chunk > 0 && (span == 0 || chunk < span)) span = chunk;
-    const int nw = span > 0 ? ((span + 31) / 32 < 16 ? (span + 31) / 32 : 16) : 8;
+    const int nw = span > 0 ? ((span + 31) / 32 < 16 ? (span + 31) / 32 : 16) : 16;
     dim3 grid((unsigned)((long)rows * heads));
     const size_t smem = (size_t)(((maps * D + 3) & ~3) + nw * maps * (Dv + 2) + (maps > 1 ? ((Dv + 3) & ~3) + 32 : 0)) * sizeof(float);
     if (smem > 48 * 1024 || (long)rows * heads > 0x7fffffffL) return CML_ERR_BAD_SIZE;

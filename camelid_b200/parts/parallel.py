@@ -95,6 +95,9 @@ class ParallelMixers(Part):
     def query_tile_sizes(self):
         return [r for b in self.branches for r in b.query_tile_sizes()]
 
+    def workspace_per_row(self):
+        return sum(b.workspace_per_row() for b in self.branches)
+
     def _projections(self, ctx, x):
         """Every branch's columns of the stacked input product (None each where there is no such product): complete rows, or
         split sums on one-token steps where every branch takes those."""

@@ -237,3 +237,16 @@ def test_benchmark_counts_every_matrix_once():
         assert bytes_step["weights"] == 2 * want
         assert 0.98 < bytes_step["weights"] / b.kizezen_step_bytes(other, 8, 512.0, 2)["weights"] < 1.02
         assert 0.9 < b.zabunex_prefill_flops(cfg, 2048) / b.kizezen_prefill_flops(other, 2048) < 1.1
+
+
+def test_memory_plan_counts_states_and_the_chunks_scratch():
+    from zabunex_models import WIDE
+    model = DecoderModel.from_config(WIDE, dtype=torch.bfloat16, device="cpu")
+    part = model.blocks[0].mixer.branches[1]
+    assert part.workspace_per_row() >= 4 * (part.in_width + 2 * 64 + 4 * 32 * 64 // 64)
+    plan, more = model.memory_plan(4096, 4, 2048), model.memory_plan(4096, 5, 2048)
+    assert model.blocks[0].mixer.workspace_per_row() == part.workspace_per_row()             # through the mixers side by side
+    assert plan.workspace > 2048 * part.workspace_per_row()
+    states = 4 * 32 * 64 + 3 * (128 + 256) + 2 * 64 * 128 + 3 * (128 + 256)          # S and the kept inputs of both parallel layers' right sides
+    kept = 3 * (256 + 128 + 256) + 2 * (384 + 128 + 64)                              # and of their left sides
+    assert more.cache - plan.cache == 4 * (states + kept)
