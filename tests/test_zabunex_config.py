@@ -78,7 +78,7 @@ def test_weights_side_by_side():
     assert torch.equal(model.blocks[1].mixer.sink_w, torch.zeros(4))
 
 
-@pytest.mark.parametrize("rows,largest", [(32, 240), (4, 17), (6, 200.5), (2, 9), (10, 300), (30, 16), (7, 50)])
+@pytest.mark.parametrize("rows,largest", [(32, 250), (4, 17), (6, 200.5), (2, 9), (10, 300), (30, 16), (7, 50)])
 def test_the_bias_table_written_out_by_distance(rows, largest):
     table = distance_buckets(rows, largest)
     assert table == [pz.bucket(d, rows, largest) for d in range(len(table))]
@@ -248,5 +248,5 @@ def test_memory_plan_counts_states_and_the_chunks_scratch():
     assert model.blocks[0].mixer.workspace_per_row() == part.workspace_per_row()             # through the mixers side by side
     assert plan.workspace > 2048 * part.workspace_per_row()
     states = 4 * 32 * 64 + 3 * (128 + 256) + 2 * 64 * 128 + 3 * (128 + 256)          # S and the kept inputs of both parallel layers' right sides
-    kept = 3 * (256 + 128 + 256) + 2 * (384 + 128 + 64)                              # and of their left sides
+    kept = 3 * (384 + 128 + 256) + 2 * (384 + 128 + 64)                              # and of their left sides
     assert more.cache - plan.cache == 4 * (states + kept)

@@ -64,8 +64,8 @@ ODD = config(44, 61, [
 # sizes of the tensor-core kernels: heads of 64 and 128 channels (equal and unlike values), blocks of 130 and 200 positions, states of
 # 64 and 128 channels
 WIDE = config(128, 83, [
-    layer(parallel(left(4, 2, 64, 128, 4, 130, 0.125, (32, 10000.0, 2.0)), right(4, 32, 64, 2, 4, 2), 0.9, 0.8), 256),
-    layer(attention(4, 2, 64, 0.125, 128, (0.3, 100)), 192),
+    layer(parallel(left(6, 2, 64, 128, 4, 130, 0.13, (32, 10000.0, 2.0)), right(4, 32, 64, 2, 4, 2), 0.9, 0.8), 256),
+    layer(attention(6, 3, 64, 0.12, 128, (0.3, 100)), 192),
     layer(attention(2, 2, 128, 0.1, 250, (0.1, 64)), 136),
     layer(parallel(left(3, 1, 128, 64, 3, 200, 0.09, (128, 500000.0, 8.0)), right(2, 64, 128, 1, 4, 1), 1.2, 0.5), 320),
 ])
